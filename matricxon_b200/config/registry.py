@@ -125,6 +125,14 @@ def _register_builtin() -> None:
         config_class=KefasunConfig,
         build_model=_build_decoder,
     ))
+    from matricxon_b200.config.seredra import SeredraConfig
+
+    register_architecture(ArchitectureEntry(
+        name="Seredra",
+        aliases=("seredra",),
+        config_class=SeredraConfig,
+        build_model=_build_decoder,
+    ))
 
 
 _register_builtin()

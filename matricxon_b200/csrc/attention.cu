@@ -5,7 +5,8 @@
 // the query at absolute position p sees key j iff j <= p and (window == 0 or j > p - window or j < keep_first):
 // a window may keep the sequence's first `keep_first` tokens in sight for good (0: none); they keep their
 // true positions, and the chunks between them and the window are skipped, not masked.
-// Scores are q.k * scale, softmax is max-subtracted, query head h reads KV head h / (heads / kv heads)
+// Scores are q.k * scale (capped, then less a distance bias where the caller asks: r1_h ln(1 + r2_h (p - j)), a
+// pair of numbers per query head), softmax is max-subtracted, query head h reads KV head h / (heads / kv heads)
 // (app/native/src/mx_attention.c:16-68). Scores, softmax and the weighted sum are float whatever T is.
 //
 // One block handles (query token, KV head, group of up to 16 query heads, key split). Keys are
@@ -45,6 +46,7 @@ struct AttnParams {
     float softcap;            // > 0: scores become softcap * tanh(score / softcap) before the softmax
     const float* sink;        // [n_heads] or null: exp(sink[h]) joins the softmax's denominator, with no value
     int keep_first;           // with a window: keys j < keep_first stay visible whatever the distance
+    const float* distance;    // [2][n_heads] (r1, then r2) or null: scores lose r1 ln(1 + r2 (p - j))
 };
 
 template <typename T> struct Vec16;  // 16 bytes of T
@@ -219,6 +221,9 @@ paged_attention_kernel(const AttnParams p) {
                 if (h < gc) {
                     float sv = s[hs] * p.scale;
                     if (p.softcap > 0.f) sv = p.softcap * tanhf(sv / p.softcap);
+                    if (p.distance && valid)
+                        sv -= p.distance[head0 + h] *
+                              logf(fmaf(p.distance[p.n_heads + head0 + h], (float)(pos - kpos), 1.f));
                     sv = valid ? sv : -INFINITY;
                     const float m_new = fmaxf(m_run[hs], warp_max(sv));
                     const float pj = valid ? expf(sv - m_new) : 0.f;
@@ -489,7 +494,7 @@ extern "C" int mx_paged_attention(const void* q, int dtype, int q_stride, const 
                                   int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                   int window, float scale, void* out, int out_stride,
                                   int n_splits, float* scratch, int* status, float softcap, const float* sink,
-                                  int keep_first, cudaStream_t stream) {
+                                  int keep_first, const float* distance, cudaStream_t stream) {
     if (n_tokens <= 0) return MX_OK;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0)
         MX_REFUSE("attention: %d heads are not a multiple of %d kv heads", n_heads, n_kv_heads);
@@ -510,6 +515,7 @@ extern "C" int mx_paged_attention(const void* q, int dtype, int q_stride, const 
     p.window = window; p.n_splits = n_splits; p.scale = scale;
     p.softcap = softcap; p.sink = sink;
     p.keep_first = window > 0 ? max(keep_first, 0) : 0;
+    p.distance = distance;
     const bool two = head_dim > ATT_THREADS;
     if (dtype == MX_DTYPE_F32)
         return two ? launch_attention<float, 2>(p, n_tokens, stream) : launch_attention<float, 1>(p, n_tokens, stream);
@@ -600,5 +606,5 @@ extern "C" int mx_paged_attention_static(const void* q, int dtype, int q_stride,
     if (rc != MX_OK) return rc;
     return mx_paged_attention(q, dtype, q_stride, cache, n_pages, page_size, block_tables, bt_stride,
                               tok_seq, positions, n_tokens, n_heads, n_kv_heads, head_dim, window,
-                              scale, out, out_stride, n_splits, scratch, status, 0.f, nullptr, 0, stream);
+                              scale, out, out_stride, n_splits, scratch, status, 0.f, nullptr, 0, nullptr, stream);
 }

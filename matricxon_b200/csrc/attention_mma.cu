@@ -1,7 +1,8 @@
 // Tensor-core paged attention for bfloat16: prompt portions and decode tokens.
 //
 // Same mathematics and visibility rule as attention.cu (query at p sees key j iff j <= p and
-// (window == 0 or j > p - window or j < keep_first); scores q.k * scale; float softmax; query head h reads KV
+// (window == 0 or j > p - window or j < keep_first); scores q.k * scale, optionally capped or less a distance bias
+// r1_h ln(1 + r2_h (p - j)); float softmax; query head h reads KV
 // head h / group), cf. app/native/src/mx_attention.c:16-68 and
 // app/architectures/qwen_layers.py:12-17,94-100.
 //
@@ -72,6 +73,7 @@ struct MmaAttnParams {
     // (cap_in = scale / cap), already in the units of the exponential; 0: no cap
     float cap_log2, cap_in;
     const float* sink;           // [heads] or null: exp(sink[h]) joins the softmax's denominator, with no value
+    const float* distance;       // [2][heads] (r1, then r2) or null: scores lose r1 ln(1 + r2 (p - j))
 };
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], unsigned a0, unsigned a1, unsigned a2,
@@ -186,7 +188,7 @@ __device__ __forceinline__ void issue_chunk(const MmaAttnParams& p, __nv_bfloat1
 struct One { static constexpr int value = 1; };
 struct Two { static constexpr int value = 2; };
 
-template <int HD, bool NARROW>
+template <int HD, bool NARROW, bool BIASED>
 __global__ void __launch_bounds__(NARROW ? NARROW_THREADS : MMA_THREADS, NARROW ? 1 : 3)
 attention_mma_kernel(const MmaAttnParams p) {
     constexpr int KB = HD / 32;                 // 32-wide blocks of the head dim
@@ -242,6 +244,14 @@ attention_mma_kernel(const MmaAttnParams p) {
         r_head[i] = rr - r_tok[i] * group;
         r_pos[i] = ctx + r_tok[i];
         r_lo[i] = first_visible_key(r_pos[i], p.window);
+    }
+    float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};    // distance bias of the row's head, in log2 units as it stands
+    if (BIASED) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            r1[i] = p.distance[kh * group + r_head[i]];
+            r2[i] = p.distance[p.n_heads + kh * group + r_head[i]];
+        }
     }
     // key range of the block (what is fetched) and of the warp (what it computes)
     const int hi_tile = ctx + tile_last / group;
@@ -337,7 +347,8 @@ attention_mma_kernel(const MmaAttnParams p) {
                 for (int b = 0; b < 4; ++b)
                     mma_bf16(s[ch][b], qf[0][kb].z, qf[1][kb].z, qf[0][kb].w, qf[1][kb].w, kf[b].z, kf[b].w);
             }
-        const float scale_log2 = p.cap_log2 > 0.f ? 1.f : p.scale_log2;
+        const bool in_units = p.cap_log2 > 0.f || BIASED;     // scores already in units of the exponential
+        const float scale_log2 = in_units ? 1.f : p.scale_log2;
         if (p.cap_log2 > 0.f) {
             // small arguments (the usual case) take the polynomial; one large score in the warp's chunk sends
             // the whole warp through the exponential form
@@ -366,6 +377,24 @@ attention_mma_kernel(const MmaAttnParams p) {
 #pragma unroll
                         for (int e = 0; e < 4; ++e) s[ch][b][e] = p.cap_log2 * tanh_by_exp2(s[ch][b][e]);
             }
+        }
+        if (BIASED) {
+            // 1 + r2 (p - j) = (1 + r2 (p - first key of this thread)) - r2 * (key - first): keys beyond p give a
+            // logarithm of nothing, which the mask below throws away
+            const float to_units = p.cap_log2 > 0.f ? 1.f : p.scale_log2;
+#pragma unroll
+            for (int ch = 0; ch < NCH; ++ch)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const float base = fmaf(r2[i], (float)(r_pos[i] - first_key[ch] - 8 * t), 1.f);
+#pragma unroll
+                    for (int b = 0; b < 4; ++b)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) {
+                            const float away = fmaf(r2[i], -(float)(2 * b + e), base);
+                            s[ch][b][2 * i + e] = fmaf(s[ch][b][2 * i + e], to_units, -r1[i] * fast_log2(away));
+                        }
+                }
         }
         // mask (only where the chunks cross an edge), running max and sum for rows g, g + 8
         float m_new[2] = {m_run[0], m_run[1]};
@@ -650,8 +679,8 @@ attention_mma_kernel(const MmaAttnParams p) {
     }
 }
 
-template <int HD, bool NARROW>
-int launch_mma(const MmaAttnParams& p, cudaStream_t stream) {
+template <int HD, bool NARROW, bool BIASED>
+int launch_mma_kernel(const MmaAttnParams& p, cudaStream_t stream) {
     const size_t stage_bytes = 2 * (size_t)CHUNK * HD * sizeof(__nv_bfloat16);
     size_t smem = stage_bytes * (NARROW ? NARROW_STAGES * NARROW_WARPS : WIDE_STAGES);
     if (NARROW) {
@@ -659,13 +688,18 @@ int launch_mma(const MmaAttnParams& p, cudaStream_t stream) {
         if (reduce > smem) smem = reduce;
     }
     if (smem + 1024 > 48 * 1024) {   // the kernel also has a little static shared memory
-        cudaError_t e = cudaFuncSetAttribute(attention_mma_kernel<HD, NARROW>,
+        cudaError_t e = cudaFuncSetAttribute(attention_mma_kernel<HD, NARROW, BIASED>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) MX_REFUSE("attention: cannot reserve %zu bytes of shared memory", smem);
     }
     dim3 grid(p.n_tiles, p.n_kv_heads, p.n_splits);
-    mx_launch_chained(attention_mma_kernel<HD, NARROW>, grid, dim3(NARROW ? NARROW_THREADS : MMA_THREADS), smem, stream, p);
+    mx_launch_chained(attention_mma_kernel<HD, NARROW, BIASED>, grid, dim3(NARROW ? NARROW_THREADS : MMA_THREADS), smem, stream, p);
     return mx_launch_status();
+}
+
+template <int HD, bool NARROW>
+int launch_mma(const MmaAttnParams& p, cudaStream_t stream) {
+    return p.distance ? launch_mma_kernel<HD, NARROW, true>(p, stream) : launch_mma_kernel<HD, NARROW, false>(p, stream);
 }
 
 }  // namespace
@@ -683,7 +717,7 @@ extern "C" int mx_paged_attention_mma(const void* q, int q_stride, const void* c
                                       int n_heads, int n_kv_heads, int head_dim, int window,
                                       float scale, void* out, int out_stride, int n_splits,
                                       float* scratch, int* status, float softcap, const float* sink,
-                                      int keep_first, cudaStream_t stream) {
+                                      int keep_first, const float* distance, cudaStream_t stream) {
     if (n_tiles <= 0 || n_tokens <= 0) return MX_OK;
     if (n_kv_heads <= 0 || n_heads % n_kv_heads != 0)
         MX_REFUSE("attention: %d heads are not a multiple of %d kv heads", n_heads, n_kv_heads);
@@ -710,6 +744,7 @@ extern "C" int mx_paged_attention_mma(const void* q, int q_stride, const void* c
     p.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
     p.sink = sink;
+    p.distance = distance;
     int rc;
     if (head_dim == 64) rc = narrow ? launch_mma<64, true>(p, stream) : launch_mma<64, false>(p, stream);
     else rc = narrow ? launch_mma<128, true>(p, stream) : launch_mma<128, false>(p, stream);

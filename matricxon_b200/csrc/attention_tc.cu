@@ -3,7 +3,8 @@
 //
 // Same mathematics and visibility rule as attention.cu / attention_mma.cu (query at p sees key j
 // iff j <= p and (window == 0 or j > p - window or j < keep: the sequence's first `keep` positions stay in
-// sight under a window); scores q.k * scale; float softmax; query head h
+// sight under a window); scores q.k * scale, optionally capped or less a distance bias r1_h ln(1 + r2_h (p - j));
+// float softmax; query head h
 // reads KV head h / group), cf. app/native/src/mx_attention.c:16-68 and
 // app/architectures/qwen_layers.py:12-17,94-100.
 //
@@ -87,6 +88,7 @@ struct AtParams {
     // (cap_in = scale / cap), already in the units of the exponential; 0: no cap
     float cap_log2, cap_in;
     const float* sink;           // [heads] or null: exp(sink[h]) joins the softmax's denominator, with no value
+    const float* distance;       // [2][heads] (r1, then r2) or null: scores lose r1 ln(1 + r2 (p - j))
 };
 
 __device__ __forceinline__ unsigned smem_u32(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -225,6 +227,7 @@ __device__ __forceinline__ unsigned at_pack(float lo, float hi) {
     return *reinterpret_cast<unsigned*>(&v);
 }
 
+template <bool BIASED>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                     const __grid_constant__ CUtensorMap v_map, const AtParams p) {
@@ -453,6 +456,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
         const int pos = valid ? ctx + tok0 + t_in : -1;                 // -1: every key is masked
         const int lo = first_visible_key(pos, p.window);
         const unsigned lane_base = (unsigned)(32 * (warp & 3)) << 16;
+        // distance bias of the row's head; a row that belongs to no token takes none (its scores stay numbers)
+        const float r1 = BIASED && valid ? p.distance[kh * p.group + h_in] : 0.f;
+        const float r2 = BIASED && valid ? p.distance[p.n_heads + kh * p.group + h_in] : 0.f;
         float m_ref = -INFINITY, l_run = 0.f;
         bool alive = true;
         // Phases of the "P V done" barrier are consumed strictly in order (phase j completes when the
@@ -502,6 +508,14 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
                         for (int c = 0; c < 64; ++c) sc[c] = p.cap_log2 * tanh_by_exp2(sc[c]);
                     }
                 }
+                if (BIASED) {
+                    // in the units of the exponential; keys beyond p give a logarithm of nothing, masked below
+                    const float to_units = p.cap_log2 > 0.f ? 1.f : p.scale_log2;
+                    const float base = fmaf(r2, (float)(pos - k0), 1.f);
+#pragma unroll
+                    for (int c = 0; c < 64; ++c)
+                        sc[c] = fmaf(sc[c], to_units, -r1 * fast_log2(fmaf(r2, -(float)c, base)));
+                }
                 if (edge) {
 #pragma unroll
                     for (int c = 0; c < 64; ++c) {
@@ -525,7 +539,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_cons
                 alive = false;
                 break;                                  // all 256 threads see the flag after the barrier
             }
-            const float scale_log2 = p.cap_log2 > 0.f ? 1.f : p.scale_log2;
+            const float scale_log2 = p.cap_log2 > 0.f || BIASED ? 1.f : p.scale_log2;
             mx = fmaxf(mx, half_max[j & 1][part ^ 1][row]) * scale_log2;
             const bool jump = mx > m_ref + AT_JUMP || (m_ref == -INFINITY && mx > -INFINITY);
             const float m_new = jump ? mx : m_ref;
@@ -695,7 +709,8 @@ extern "C" int mx_paged_attention_tc_split(const void* q, int q_stride, const vo
                                            const int* context_lens, const int* tiles, int n_tiles, int n_tokens,
                                            int n_heads, int n_kv_heads, int head_dim, int window, float scale,
                                            void* out, int out_stride, int n_splits, float* scratch, int* status,
-                                           float softcap, const float* sink, int keep_first, cudaStream_t stream) {
+                                           float softcap, const float* sink, int keep_first, const float* distance,
+                                           cudaStream_t stream) {
     if (n_tiles <= 0 || n_tokens <= 0) return MX_OK;
     if (n_splits < 1 || n_splits > 64) MX_REFUSE("tcgen05 attention: %d key splits", n_splits);
     if (n_splits > 1 && scratch == nullptr) MX_REFUSE("tcgen05 attention: key splits without scratch memory");
@@ -746,17 +761,22 @@ extern "C" int mx_paged_attention_tc_split(const void* q, int q_stride, const vo
     p.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
     p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
     p.sink = sink;
+    p.distance = distance;
     p.n_splits = n_splits;
     p.part_o = scratch;
     p.part_ml = scratch ? scratch + (size_t)n_tokens * n_heads * n_splits * AT_HD : nullptr;
     const size_t smem = (size_t)(2 + 2 * AT_STAGES * 2) * AT_TILE + 1024;
     static bool attribute_set = false;
     if (!attribute_set) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(attention_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) MX_REFUSE("tcgen05 attention: cannot reserve %zu bytes of shared memory", smem);
         attribute_set = true;
     }
-    attention_tc_kernel<<<dim3(n_tiles, n_kv_heads, n_splits), AT_THREADS, smem, stream>>>(q_map, k_map, v_map, p);
+    const dim3 grid(n_tiles, n_kv_heads, n_splits);
+    if (distance) attention_tc_kernel<true><<<grid, AT_THREADS, smem, stream>>>(q_map, k_map, v_map, p);
+    else attention_tc_kernel<false><<<grid, AT_THREADS, smem, stream>>>(q_map, k_map, v_map, p);
     const int rc = mx_launch_status();
     if (rc != MX_OK || n_splits == 1) return rc;
     return mx_attention_merge_bf16_sink(p.part_o, p.part_ml, out, out_stride, n_tokens, n_heads, AT_HD, n_splits, sink,
@@ -770,5 +790,5 @@ extern "C" int mx_paged_attention_tc(const void* q, int q_stride, const void* ca
                                      void* out, int out_stride, int* status, cudaStream_t stream) {
     return mx_paged_attention_tc_split(q, q_stride, cache, n_pages, page_size, block_tables, bt_stride, cu_q,
                                        context_lens, tiles, n_tiles, n_tokens, n_heads, n_kv_heads, head_dim, window,
-                                       scale, out, out_stride, 1, nullptr, status, 0.f, nullptr, 0, stream);
+                                       scale, out, out_stride, 1, nullptr, status, 0.f, nullptr, 0, nullptr, stream);
 }

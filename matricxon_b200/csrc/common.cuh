@@ -134,6 +134,12 @@ __device__ __forceinline__ float tanh_by_exp2(float x) {
     return 1.f - __fdividef(2.f, 1.f + e);
 }
 
+__device__ __forceinline__ float fast_log2(float x) {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // tanh of a small argument on the FMA pipe: the odd Taylor polynomial up to x^11, whose first dropped term is
 // below 2e-8 of x for |x| <= TANH_SMALL. Scores under a cap are mostly that small (|score| <= 0.35 cap), and the
 // special-function units that tanh_by_exp2 needs are what bounds a softmax.
@@ -153,6 +159,18 @@ __device__ __forceinline__ float gelu_tanh(float u) {
     const float k0 = 0.7978845608028654f, k1 = 0.044715f;
     return 0.5f * u * (1.f + tanhf(k0 * (u + k1 * u * u * u)));
 }
+// Epilogue modes of every matrix product, with v = acc + bias: 0 out(T) = v; 1 out(T) = gelu_tanh(v);
+// 2 out(f32) = residual + v; 3 out(f32) = v; 4 out(T) = max(v, 0)^2.
+#define MX_MODE_NONE 0
+#define MX_MODE_GELU 1
+#define MX_MODE_RESIDUAL 2
+#define MX_MODE_F32 3
+#define MX_MODE_RELU2 4
+#define MX_MODE_LAST 4
+__host__ __device__ __forceinline__ bool mx_mode_is_float(int mode) {
+    return mode == MX_MODE_RESIDUAL || mode == MX_MODE_F32;
+}
+
 // The same with the hardware tanh (relative error about 2^-11): for results that are rounded to
 // bfloat16 (2^-9) right after; the 32-bit path keeps tanhf.
 __device__ __forceinline__ float gelu_tanh_fast(float u) {
@@ -160,4 +178,17 @@ __device__ __forceinline__ float gelu_tanh_fast(float u) {
     float t;
     asm("tanh.approx.f32 %0, %1;\n" : "=f"(t) : "f"(k0 * (u + k1 * u * u * u)));
     return 0.5f * u * (1.f + t);
+}
+
+// The activation that an epilogue mode puts on a value (modes without one return it): exact, and with the hardware
+// tanh for results that are rounded to bfloat16.
+__device__ __forceinline__ float relu_squared(float v) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+}
+__device__ __forceinline__ float mode_activation(float v, int mode) {
+    return mode == MX_MODE_GELU ? gelu_tanh(v) : (mode == MX_MODE_RELU2 ? relu_squared(v) : v);
+}
+__device__ __forceinline__ float mode_activation_fast(float v, int mode) {
+    return mode == MX_MODE_GELU ? gelu_tanh_fast(v) : (mode == MX_MODE_RELU2 ? relu_squared(v) : v);
 }

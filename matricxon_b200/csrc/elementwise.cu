@@ -568,6 +568,7 @@ extern "C" int mx_rope_kv_write(void* qkv, int dtype, int row_stride, const int*
 // mode 1: out(T)  = gelu_tanh(acc + bias)
 // mode 2: out(f32) = residual + acc + bias     (out may alias residual)
 // mode 3: out(f32) = acc + bias
+// mode 4: out(T)  = max(acc + bias, 0)^2
 template <typename TAcc, typename TOut>
 __global__ void epilogue_kernel(const TAcc* __restrict__ acc, const float* __restrict__ bias,
                                 const float* residual, TOut* out, long long total, int n_cols,
@@ -576,7 +577,7 @@ __global__ void epilogue_kernel(const TAcc* __restrict__ acc, const float* __res
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
         float v = to_float(acc[i]);
         if (bias) v += bias[(int)(i % n_cols)];
-        if (mode == 1) v = gelu_tanh(v);
+        v = mode_activation(v, mode);
         if (mode == 2) v += residual[i];
         out[i] = from_float<TOut>(v);
     }
@@ -621,6 +622,10 @@ __global__ void epilogue_vec_kernel(const TAcc* __restrict__ acc, const float* _
 #pragma unroll
             for (int e = 0; e < 4; ++e) v[k][e] = sizeof(TOut) == 4 ? gelu_tanh(v[k][e]) : gelu_tanh_fast(v[k][e]);
         }
+        if (mode == MX_MODE_RELU2) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[k][e] = relu_squared(v[k][e]);
+        }
         if (mode == 2) { v[k][0] += r[k].x; v[k][1] += r[k].y; v[k][2] += r[k].z; v[k][3] += r[k].w; }
         if (sizeof(TOut) == 4) {
             *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + at) = make_float4(v[k][0], v[k][1], v[k][2], v[k][3]);
@@ -639,7 +644,7 @@ extern "C" int mx_epilogue(const void* acc, int acc_dtype, const float* bias, co
                            cudaStream_t stream) {
     const long long total = n_rows * n_cols;
     if (total <= 0) return MX_OK;
-    if (mode < 0 || mode > 3) MX_REFUSE("epilogue: unknown mode %d", mode);
+    if (mode < 0 || mode > MX_MODE_LAST) MX_REFUSE("epilogue: unknown mode %d", mode);
     if (mode == 2 && residual == nullptr) MX_REFUSE("epilogue: residual mode without a residual");
     const int threads = 256;
     const bool aligned = ((reinterpret_cast<uintptr_t>(acc) | reinterpret_cast<uintptr_t>(bias) |

@@ -8,7 +8,7 @@
 // app/architectures/starcoder2_layers.py:19-23).
 //
 // Epilogue modes: 0 out(T) = v; 1 out(T) = gelu_tanh(v); 2 out(f32) = residual + v;
-// 3 out(f32) = v, where v = acc + bias.
+// 3 out(f32) = v; 4 out(T) = max(v, 0)^2, where v = acc + bias.
 #include "common.cuh"
 
 namespace {
@@ -75,7 +75,7 @@ gemm_simt_kernel(const TIn* __restrict__ A, const TIn* __restrict__ W,
             if (n >= N) continue;
             float v = acc[i][j];
             if (bias) v += bias[n];
-            if (mode == 1) v = gelu_tanh(v);
+            v = mode_activation(v, mode);
             const size_t o = (size_t)m * ldo + n;
             if (mode == 2) v += residual[o];
             out[o] = from_float<TOut>(v);
@@ -90,9 +90,9 @@ extern "C" int mx_gemm_simt(const void* A, const void* W, int in_dtype, const fl
                             int lda, int ldw, int ldo, int mode, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return MX_OK;
     if (K <= 0) MX_REFUSE("gemm: K must be positive, got %d", K);
-    if (mode < 0 || mode > 3) MX_REFUSE("gemm: unknown epilogue mode %d", mode);
+    if (mode < 0 || mode > MX_MODE_LAST) MX_REFUSE("gemm: unknown epilogue mode %d", mode);
     if (mode == 2 && residual == nullptr) MX_REFUSE("gemm: residual mode without a residual");
-    const int expected_out = (mode >= 2 || in_dtype == MX_DTYPE_F32) ? MX_DTYPE_F32 : MX_DTYPE_BF16;
+    const int expected_out = (mx_mode_is_float(mode) || in_dtype == MX_DTYPE_F32) ? MX_DTYPE_F32 : MX_DTYPE_BF16;
     if (out_dtype != expected_out)
         MX_REFUSE("gemm: epilogue mode %d with input dtype %d writes dtype %d, not %d", mode,
                   in_dtype, expected_out, out_dtype);

@@ -15,7 +15,7 @@
 // (app/architectures/qwen_layers.py:50-53, app/architectures/starcoder2_layers.py:19-23).
 //
 // Epilogue modes as in gemm_simt.cu: 0 out(bf16) = v; 1 out(bf16) = gelu_tanh(v);
-// 2 out(f32) = residual + v; 3 out(f32) = v, with v = acc + bias.
+// 2 out(f32) = residual + v; 3 out(f32) = v; 4 out(bf16) = max(v, 0)^2, with v = acc + bias.
 #include <cooperative_groups.h>
 
 #include "common.cuh"
@@ -267,9 +267,9 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const __nv_bflo
         if (n >= N || m >= M) continue;
         float v = total(f, m);
         if (bias) v += bias[n];
-        if (mode == 1) v = gelu_tanh_fast(v);
+        v = mode_activation_fast(v, mode);
         const size_t o = (size_t)m * ldo + n;
-        if (mode >= 2) {
+        if (mx_mode_is_float(mode)) {
             if (mode == 2) v += residual[o];
             reinterpret_cast<float*>(out)[o] = v;
         } else {
@@ -316,9 +316,9 @@ extern "C" int mx_gemm_skinny(const void* x, const void* W, const float* bias, c
     if (M <= 0 || N <= 0) return MX_OK;
     const int rc = check_skinny(M, K, ldx, ldw);
     if (rc != MX_OK) return rc;
-    if (mode < 0 || mode > 3) MX_REFUSE("skinny gemm: unknown epilogue mode %d", mode);
+    if (mode < 0 || mode > MX_MODE_LAST) MX_REFUSE("skinny gemm: unknown epilogue mode %d", mode);
     if (mode == 2 && residual == nullptr) MX_REFUSE("skinny gemm: residual mode without a residual");
-    if ((mode >= 2) != (out_dtype == MX_DTYPE_F32))
+    if (mx_mode_is_float(mode) != (out_dtype == MX_DTYPE_F32))
         MX_REFUSE("skinny gemm: epilogue mode %d does not write dtype %d", mode, out_dtype);
     const SkinnyRope none = {};
     const int grid = (N + 15) / 16;

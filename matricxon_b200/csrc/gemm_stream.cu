@@ -31,7 +31,7 @@
 // moves on, so the block always reaches the point where tensor memory is freed.
 //
 // Epilogue modes as in gemm_simt.cu: 0 out(bf16) = v; 1 out(bf16) = gelu_tanh(v);
-// 2 out(f32) = residual + v; 3 out(f32) = v, with v = acc + bias.
+// 2 out(f32) = residual + v; 3 out(f32) = v; 4 out(bf16) = max(v, 0)^2, with v = acc + bias.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -221,7 +221,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_const
                         for (int j = 0; j < 16; ++j) {
                             if (c0 + j >= M) break;
                             float v = __uint_as_float(r[j]) + b;
-                            if (mode == 1) v = gelu_tanh_fast(v);
+                            v = mode_activation_fast(v, mode);
                             reinterpret_cast<__nv_bfloat16*>(out)[(size_t)(c0 + j) * ldo + n] = __float2bfloat16_rn(v);
                         }
                     }
@@ -269,9 +269,9 @@ extern "C" int mx_gemm_stream(const void* x, const void* W, const float* bias, c
     if (ldx % 8 != 0 || ldw % 8 != 0) MX_REFUSE("streaming gemm: row strides %d, %d are not multiples of 8", ldx, ldw);
     if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(W)) & 15)
         MX_REFUSE("streaming gemm: operands must start on 16-byte boundaries");
-    if (mode < 0 || mode > 3) MX_REFUSE("streaming gemm: unknown epilogue mode %d", mode);
+    if (mode < 0 || mode > MX_MODE_LAST) MX_REFUSE("streaming gemm: unknown epilogue mode %d", mode);
     if (mode == 2 && residual == nullptr) MX_REFUSE("streaming gemm: residual mode without a residual");
-    if ((mode >= 2) != (out_dtype == MX_DTYPE_F32))
+    if (mx_mode_is_float(mode) != (out_dtype == MX_DTYPE_F32))
         MX_REFUSE("streaming gemm: epilogue mode %d does not write dtype %d", mode, out_dtype);
     if (status == nullptr) MX_REFUSE("streaming gemm: a status word is needed for its bounded waits");
 

@@ -29,7 +29,7 @@
 // 512-row tiles on pairs of SMs (cta_group::2); mx_gemm_tcgen05 picks by the number of rows.
 //
 // Epilogue modes as in gemm_simt.cu: 0 out(bf16) = v; 1 out(bf16) = gelu_tanh(v);
-// 2 out(f32) = residual + v; 3 out(f32) = v, with v = acc + bias.
+// 2 out(f32) = residual + v; 3 out(f32) = v; 4 out(bf16) = max(v, 0)^2, with v = acc + bias.
 #include <cuda.h>
 
 #include <cstdlib>
@@ -58,7 +58,7 @@ struct TcShared {
 __device__ __forceinline__ void store_piece(const unsigned (&r)[16], const float* __restrict__ bias,
                                             const float* residual, void* out, size_t obase, int nbase, int N,
                                             int mode) {
-    if (mode >= 2) {
+    if (mx_mode_is_float(mode)) {
         float* o = reinterpret_cast<float*>(out) + obase;
         const float* res = (mode == 2) ? residual + obase : nullptr;
         if (nbase + 16 <= N && (obase % 4) == 0) {
@@ -97,7 +97,7 @@ __device__ __forceinline__ void store_piece(const unsigned (&r)[16], const float
             for (int e = 0; e < 8; ++e) {
                 v[e] = __uint_as_float(r[j + e]);
                 if (bias) v[e] += bias[nbase + j + e];
-                if (mode == 1) v[e] = gelu_tanh_fast(v[e]);
+                v[e] = mode_activation_fast(v[e], mode);
             }
             uint4 pk;
             __nv_bfloat162 h0 = __floats2bfloat162_rn(v[0], v[1]);
@@ -113,7 +113,7 @@ __device__ __forceinline__ void store_piece(const unsigned (&r)[16], const float
             if (nbase + j >= N) break;
             float v = __uint_as_float(r[j]);
             if (bias) v += bias[nbase + j];
-            if (mode == 1) v = gelu_tanh_fast(v);
+            v = mode_activation_fast(v, mode);
             o[j] = __float2bfloat16_rn(v);
         }
     }
@@ -268,6 +268,9 @@ struct EpilogueLane {
                         if (mode == 1) {
                             v[i].x = gelu_tanh_fast(v[i].x); v[i].y = gelu_tanh_fast(v[i].y);
                             v[i].z = gelu_tanh_fast(v[i].z); v[i].w = gelu_tanh_fast(v[i].w);
+                        } else if (mode == MX_MODE_RELU2) {
+                            v[i].x = relu_squared(v[i].x); v[i].y = relu_squared(v[i].y);
+                            v[i].z = relu_squared(v[i].z); v[i].w = relu_squared(v[i].w);
                         }
                         __nv_bfloat162 lo = __floats2bfloat162_rn(v[i].x, v[i].y);
                         __nv_bfloat162 hi = __floats2bfloat162_rn(v[i].z, v[i].w);
@@ -310,7 +313,7 @@ struct EpilogueLane {
                     else *dst = (mode == 2 ? residual[at] : 0.f) + v[e];
                 } else {
                     reinterpret_cast<__nv_bfloat16*>(out)[at] =
-                        __float2bfloat16_rn(mode == 1 ? gelu_tanh_fast(v[e]) : v[e]);
+                        __float2bfloat16_rn(mode_activation_fast(v[e], mode));
                 }
             }
         }
@@ -1032,14 +1035,14 @@ extern "C" int mx_gemm_tcgen05(const void* A, const void* W, const float* bias, 
         MX_REFUSE("tcgen05 gemm: row strides %d, %d are not multiples of 8 elements (16 bytes)", lda, ldw);
     if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) % 16 != 0)
         MX_REFUSE("tcgen05 gemm: operands must start on 16-byte boundaries");
-    if (mode < 0 || mode > 3) MX_REFUSE("tcgen05 gemm: unknown epilogue mode %d", mode);
+    if (mode < 0 || mode > MX_MODE_LAST) MX_REFUSE("tcgen05 gemm: unknown epilogue mode %d", mode);
     if (mode == 2 && residual == nullptr) MX_REFUSE("tcgen05 gemm: residual mode without a residual");
-    if ((mode >= 2) != (out_dtype == MX_DTYPE_F32))
+    if (mx_mode_is_float(mode) != (out_dtype == MX_DTYPE_F32))
         MX_REFUSE("tcgen05 gemm: epilogue mode %d does not write dtype %d", mode, out_dtype);
     if (status == nullptr) MX_REFUSE("tcgen05 gemm: needs a status word for its bounded waits");
     const int n_sm = sm_count();
     const int n_pairs = pair_count();
-    const bool f32_out = mode >= 2;
+    const bool f32_out = mx_mode_is_float(mode);
     // the epilogue of the 256- and 512-row kernels moves 16-byte units (8 bytes of bfloat16 outputs)
     const bool vector_ok = (ldo * (f32_out ? 4 : 2)) % (f32_out ? 16 : 8) == 0 &&
                            reinterpret_cast<uintptr_t>(out) % 16 == 0 &&

@@ -16,8 +16,12 @@
 //   registers before it computes the current one, and the shares of an output are added up once a round.
 //   q is scaled by `q_scale` on its way in. Columns of a state are independent of one another, so cutting vdim
 //   into blocks changes no number.
+//   mx_retention_scan is the same recurrence with one constant decay per head (a_t = decay_h for every channel and
+//   token), which then takes no operand; it may rotate q and k on their way in (pairs (i, i + rot/2), angle
+//   position * freq[i] in float), for portions so short that rotating once per piece of 16 value columns costs less
+//   than a pass of its own. mx_rotate_heads is that pass: heads of float rows rotated in place.
 // mx_gla_norm_gate: out[t][h][e] = o[t][h][e] / sqrt(mean_e(o^2) + eps) * weight[e] * silu(gate[t][h][e]): the
-//   per-head RMS norm and the output gate, rounded once.
+//   per-head RMS norm (`weight` null: no weight) and the output gate, rounded once.
 #include <math.h>
 
 #include "common.cuh"
@@ -89,24 +93,33 @@ gla_decay_kernel(const float* __restrict__ low, int low_ld, const float* __restr
 
 // GLA_SLICES threads share a pair of columns, each with ROWS of the key channels (dim <= GLA_SLICES * ROWS);
 // GLA_TOKENS tokens are staged per round
-template <int ROWS, int GLA_SLICES, int GLA_TOKENS>
+template <int ROWS, int GLA_SLICES, int GLA_TOKENS, bool HEAD_DECAY, bool ROTATE>
 __global__ void __launch_bounds__(GLA_COLS / 2 * GLA_SLICES)
-gla_scan_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, int v_col, const float* __restrict__ decay,
-                float q_scale, float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
-                float* __restrict__ out, int n_heads, int dim, int vdim) {
+gla_scan_kernel(const float* proj, int ld, int q_col, int k_col, int v_col, const float* decay, float q_scale,
+                float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
+                float* __restrict__ out, int n_heads, int dim, int vdim, const int* __restrict__ positions,
+                const float* __restrict__ freq, int rot) {
     // a thread's ROWS channels lie side by side (four floats of padding keep the rows of neighbouring slices on
     // different banks)
     constexpr int GLA_THREADS = GLA_COLS / 2 * GLA_SLICES;
     constexpr int PAD = ROWS + 4, R4 = ROWS / 4, CH = GLA_SLICES * ROWS;
     __shared__ __align__(16) float q_s[GLA_TOKENS][GLA_SLICES][PAD], k_s[GLA_TOKENS][GLA_SLICES][PAD],
-        a_s[GLA_TOKENS][GLA_SLICES][PAD];
+        a_s[HEAD_DECAY ? 1 : GLA_TOKENS][GLA_SLICES][PAD];
     __shared__ __align__(8) float v_s[GLA_TOKENS][GLA_COLS];
     // a thread's share of every output of the round; the shares of an output are added up once a round
     // (a shuffle chain per token would be the longest wait of the loop)
     __shared__ __align__(8) float o_s[GLA_TOKENS][GLA_SLICES][GLA_COLS];
+    pdl_trigger();
     const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * GLA_COLS;
     const int t0 = cu_q[seq], t1 = cu_q[seq + 1];
-    if (t1 <= t0) return;
+    if (t1 <= t0) {
+        // a padding sequence of a fixed-size batch, whose row bears its own number: defined output, no state
+        pdl_wait();
+        if (seq >= t0)
+            for (int c = threadIdx.x; c < GLA_COLS; c += GLA_THREADS)
+                if (col0 + c < vdim) out[((size_t)seq * n_heads + head) * vdim + col0 + c] = 0.f;
+        return;
+    }
     // the eight column pairs of a slice are neighbouring lanes: a warp's state accesses are whole 64-byte row pieces,
     // its operand loads from shared memory are broadcasts
     const int tid = threadIdx.x, pair = tid & (GLA_COLS / 2 - 1), slice = tid / (GLA_COLS / 2), col = col0 + 2 * pair;
@@ -118,6 +131,11 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, in
         S0[r] = (col < vdim && i < dim) ? s_base[(size_t)i * vdim + col] : 0.f;
         S1[r] = (col + 1 < vdim && i < dim) ? s_base[(size_t)i * vdim + col + 1] : 0.f;
     }
+    const float head_decay = HEAD_DECAY ? decay[head] : 0.f;
+    // the state is what earlier steps left; the operands are the kernel's ahead
+    pdl_wait();
+    proj = after_wait(proj);
+    if (!HEAD_DECAY) decay = after_wait(decay);
     // A round's tokens travel global memory -> registers -> shared memory; the registers of the next round are
     // asked for before this round is computed, so that the recurrence never waits for global memory.
     constexpr int PER = GLA_TOKENS * CH / GLA_THREADS;             // (token, channel) items a thread stages per array
@@ -132,7 +150,15 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, in
             const float* row = proj + (size_t)(base + j) * ld + head * dim + i;
             q_r[u] = live ? row[q_col] : 0.f;
             k_r[u] = live ? row[k_col] : 0.f;
-            a_r[u] = live ? decay[((size_t)(base + j) * n_heads + head) * dim + i] : 0.f;
+            if (!HEAD_DECAY) a_r[u] = live ? decay[((size_t)(base + j) * n_heads + head) * dim + i] : 0.f;
+            if (ROTATE && live && i < rot) {
+                const int half = rot >> 1, pair = i < half ? i : i - half, away = i < half ? half : -half;
+                float sn, cs;
+                sincosf((float)positions[base + j] * freq[pair], &sn, &cs);
+                const float turn = i < half ? -sn : sn;
+                q_r[u] = fmaf(row[q_col + away], turn, q_r[u] * cs);
+                k_r[u] = fmaf(row[k_col + away], turn, k_r[u] * cs);
+            }
         }
 #pragma unroll
         for (int u = 0; u < V_PER; ++u) {
@@ -143,13 +169,13 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, in
     };
     // one token's operands of this thread, from shared memory into registers (asked for one token ahead)
     struct Operands {
-        float4 a[R4], k[R4], q[R4];
+        float4 a[HEAD_DECAY ? 1 : R4], k[R4], q[R4];
         float2 v;
     };
     auto read = [&](Operands& into, int j) {
 #pragma unroll
         for (int u = 0; u < R4; ++u) {
-            into.a[u] = *reinterpret_cast<const float4*>(&a_s[j][slice][4 * u]);
+            if (!HEAD_DECAY) into.a[u] = *reinterpret_cast<const float4*>(&a_s[j][slice][4 * u]);
             into.k[u] = *reinterpret_cast<const float4*>(&k_s[j][slice][4 * u]);
             into.q[u] = *reinterpret_cast<const float4*>(&q_s[j][slice][4 * u]);
         }
@@ -159,7 +185,8 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, in
         float o0 = 0.f, o1 = 0.f, p0 = 0.f, p1 = 0.f;
 #pragma unroll
         for (int u = 0; u < R4; ++u) {               // channels beyond dim hold zeros: no guard needed
-            const float av[4] = {now.a[u].x, now.a[u].y, now.a[u].z, now.a[u].w};
+            const float4 a4 = HEAD_DECAY ? make_float4(head_decay, head_decay, head_decay, head_decay) : now.a[HEAD_DECAY ? 0 : u];
+            const float av[4] = {a4.x, a4.y, a4.z, a4.w};
             const float kv[4] = {now.k[u].x, now.k[u].y, now.k[u].z, now.k[u].w};
             const float qv[4] = {now.q[u].x, now.q[u].y, now.q[u].z, now.q[u].w};
 #pragma unroll
@@ -186,7 +213,7 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, in
             const int item = tid + u * GLA_THREADS, j = item / CH, i = item % CH;
             q_s[j][i / ROWS][i % ROWS] = q_r[u] * q_scale;
             k_s[j][i / ROWS][i % ROWS] = k_r[u];
-            a_s[j][i / ROWS][i % ROWS] = a_r[u];
+            if (!HEAD_DECAY) a_s[j][i / ROWS][i % ROWS] = a_r[u];
         }
 #pragma unroll
         for (int u = 0; u < V_PER; ++u) {
@@ -224,11 +251,15 @@ gla_scan_kernel(const float* __restrict__ proj, int ld, int q_col, int k_col, in
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-gla_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate, int gate_ld,
+gla_norm_gate_kernel(const float* o, const float* gate, int gate_ld,
                      const float* __restrict__ weight, float eps, T* __restrict__ out, int n_heads, int vdim) {
+    pdl_trigger();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     const int h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    pdl_wait();
     if (h >= n_heads) return;
+    o = after_wait(o);
+    gate = after_wait(gate);
     const float* src = o + ((size_t)t * n_heads + h) * vdim;
     const float* g_row = gate + (size_t)t * gate_ld + h * vdim;
     constexpr int KEPT = 8;                       // up to 256 values of a head stay in registers
@@ -248,12 +279,46 @@ gla_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate
     for (int u = 0; u < KEPT; ++u) {
         const int e = lane + 32 * u;
         if (e < vdim)
-            out[((size_t)t * n_heads + h) * vdim + e] = from_float<T>(val[u] * inv * weight[e] * (g[u] / (1.0f + expf(-g[u]))));
+            out[((size_t)t * n_heads + h) * vdim + e] = from_float<T>(val[u] * inv * (weight ? weight[e] : 1.f) * (g[u] / (1.0f + expf(-g[u]))));
     }
     for (int e = lane + 32 * KEPT; e < vdim; e += 32) {
         const float gv = g_row[e];
-        out[((size_t)t * n_heads + h) * vdim + e] = from_float<T>(src[e] * inv * weight[e] * (gv / (1.0f + expf(-gv))));
+        out[((size_t)t * n_heads + h) * vdim + e] = from_float<T>(src[e] * inv * (weight ? weight[e] : 1.f) * (gv / (1.0f + expf(-gv))));
     }
+}
+
+__global__ void rotate_heads_kernel(float* rows, int ld, int col, int n_heads, int dim, int rot,
+                                    const int* __restrict__ positions, const float* __restrict__ freq) {
+    extern __shared__ float cs[];                 // cos[half], sin[half] of the token's angles
+    pdl_trigger();
+    const int t = blockIdx.x, half = rot >> 1;
+    const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * freq[i], &cs[half + i], &cs[i]);
+    __syncthreads();
+    pdl_wait();
+    float* row = after_wait(rows) + (size_t)t * ld + col;
+    for (int item = threadIdx.x; item < n_heads * half; item += blockDim.x) {
+        const int h = item / half, i = item - h * half;
+        float* p = row + (size_t)h * dim + i;
+        const float u = p[0], v = p[half];
+        p[0] = u * cs[i] - v * cs[half + i];
+        p[half] = v * cs[i] + u * cs[half + i];
+    }
+}
+
+template <bool HEAD_DECAY, bool ROTATE>
+void launch_gla_scan(const float* proj, int ld, int q_col, int k_col, int v_col, const float* decay, float q_scale,
+                     float* state, const int* cu_q, const int* state_slots, float* out, int n_seqs, int n_heads, int dim,
+                     int vdim, const int* positions, const float* freq, int rot, cudaStream_t stream) {
+    const dim3 grid(n_seqs, n_heads, (vdim + GLA_COLS - 1) / GLA_COLS);
+#define MX_GLA(ROWS, SLICES, TOKENS)                                                                                  \
+    mx_launch_chained(gla_scan_kernel<ROWS, SLICES, TOKENS, HEAD_DECAY, ROTATE>, grid, dim3(GLA_COLS / 2 * SLICES), 0, \
+                      stream, proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q, state_slots, out, n_heads,  \
+                      dim, vdim, positions, freq, rot)
+    if (dim <= 64) MX_GLA(4, 16, 16);
+    else if (dim <= 128) MX_GLA(4, 32, 8);
+    else MX_GLA(16, 16, 8);
+#undef MX_GLA
 }
 
 }  // namespace
@@ -276,27 +341,52 @@ extern "C" int mx_gla_scan(const float* proj, int ld, int q_col, int k_col, int 
     if (n_seqs <= 0) return MX_OK;
     if (dim <= 0 || dim > 256) MX_REFUSE("gated linear attention: %d key channels per head (1..256)", dim);
     if (n_heads > 65535 || vdim > 65535 * GLA_COLS) MX_REFUSE("gated linear attention: %d heads of %d values exceed the grid", n_heads, vdim);
-    const dim3 grid(n_seqs, n_heads, (vdim + GLA_COLS - 1) / GLA_COLS);
-    if (dim <= 64)
-        gla_scan_kernel<4, 16, 16><<<grid, 128, 0, stream>>>(proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q,
-                                                            state_slots, out, n_heads, dim, vdim);
-    else if (dim <= 128)
-        gla_scan_kernel<4, 32, 8><<<grid, 256, 0, stream>>>(proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q,
-                                                             state_slots, out, n_heads, dim, vdim);
+    launch_gla_scan<false, false>(proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q, state_slots, out, n_seqs,
+                                  n_heads, dim, vdim, nullptr, nullptr, 0, stream);
+    return mx_launch_status();
+}
+
+// `head_decay` [n_heads]: S_t = head_decay_h S_(t-1) + k_t v_t^T. `freq` null: q and k are taken as they are, else they
+// are rotated over their first `rot` entries on their way in.
+extern "C" int mx_retention_scan(const float* proj, int ld, int q_col, int k_col, int v_col, const float* head_decay,
+                                 float q_scale, float* state, const int* cu_q, const int* state_slots, float* out,
+                                 int n_seqs, int n_heads, int dim, int vdim, const int* positions, const float* freq,
+                                 int rot, cudaStream_t stream) {
+    if (n_seqs <= 0) return MX_OK;
+    if (dim <= 0 || dim > 256) MX_REFUSE("retention: %d key channels per head (1..256)", dim);
+    if (n_heads > 65535 || vdim > 65535 * GLA_COLS) MX_REFUSE("retention: %d heads of %d values exceed the grid", n_heads, vdim);
+    if (rot < 0 || rot % 2 != 0 || rot > dim) MX_REFUSE("retention: %d rotated entries in a head of %d", rot, dim);
+    if (freq != nullptr && rot > 0)
+        launch_gla_scan<true, true>(proj, ld, q_col, k_col, v_col, head_decay, q_scale, state, cu_q, state_slots, out,
+                                    n_seqs, n_heads, dim, vdim, positions, freq, rot, stream);
     else
-        gla_scan_kernel<16, 16, 8><<<grid, 128, 0, stream>>>(proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q,
-                                                             state_slots, out, n_heads, dim, vdim);
+        launch_gla_scan<true, false>(proj, ld, q_col, k_col, v_col, head_decay, q_scale, state, cu_q, state_slots, out,
+                                     n_seqs, n_heads, dim, vdim, nullptr, nullptr, 0, stream);
+    return mx_launch_status();
+}
+
+// n_heads heads of `dim` entries side by side from column `col` of float rows, rotated in place over their first `rot`
+// entries: (u, v) of pair (i, i + rot/2) -> (u cos a - v sin a, v cos a + u sin a), a = position * freq[i].
+extern "C" int mx_rotate_heads(float* rows, int ld, int col, int n_tokens, int n_heads, int dim, int rot,
+                               const int* positions, const float* freq, cudaStream_t stream) {
+    if (n_tokens <= 0 || n_heads <= 0 || rot <= 0) return MX_OK;
+    if (rot % 2 != 0 || rot > dim) MX_REFUSE("rotation: %d entries in a head of %d", rot, dim);
+    if (rot * (int)sizeof(float) > 48 * 1024) MX_REFUSE("rotation: %d entries are too many", rot);
+    const int threads = n_heads * (rot / 2) >= 512 ? 256 : 128;
+    mx_launch_chained(rotate_heads_kernel, dim3(n_tokens), dim3(threads), rot * sizeof(float), stream, rows, ld, col, n_heads,
+                      dim, rot, positions, freq);
     return mx_launch_status();
 }
 
 extern "C" int mx_gla_norm_gate(const float* o, const float* gate, int gate_ld, const float* weight, float eps, void* out,
                                 int dtype, int n_tokens, int n_heads, int vdim, cudaStream_t stream) {
     if (n_tokens <= 0) return MX_OK;
+    const dim3 grid(n_tokens, (n_heads + 3) / 4);
     if (dtype == MX_DTYPE_F32)
-        gla_norm_gate_kernel<float><<<dim3(n_tokens, (n_heads + 3) / 4), 128, 0, stream>>>(o, gate, gate_ld, weight, eps,
-                                                                                          (float*)out, n_heads, vdim);
+        mx_launch_chained(gla_norm_gate_kernel<float>, grid, dim3(128), 0, stream, o, gate, gate_ld, weight, eps,
+                          (float*)out, n_heads, vdim);
     else
-        gla_norm_gate_kernel<__nv_bfloat16><<<dim3(n_tokens, (n_heads + 3) / 4), 128, 0, stream>>>(
-            o, gate, gate_ld, weight, eps, (__nv_bfloat16*)out, n_heads, vdim);
+        mx_launch_chained(gla_norm_gate_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, o, gate, gate_ld, weight, eps,
+                          (__nv_bfloat16*)out, n_heads, vdim);
     return mx_launch_status();
 }

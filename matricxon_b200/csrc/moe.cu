@@ -3,7 +3,8 @@
 // mx_moe_route: per token the router's logits z = R h on the FP32 cores (R float [experts][K]), scores
 //   s = sigmoid(z), and the choice: the experts form `n_groups` runs of neighbours, a run is worth the sum of its
 //   two largest scores, only the `keep` best runs may supply experts, and of those the `top` largest scores win
-//   (ties go to the lower index). The weights are the winners' scores over their sum (+ 1e-20) times `scale`.
+//   (ties go to the lower index). The weights are the winners' scores over their sum (+ 1e-20) times `scale`, or,
+//   with `normalize` 0, the scores themselves times `scale`.
 //   The kernel also counts the pairs of every expert and gives each (token, slot) pair its place among its
 //   expert's pairs (the order inside an expert is whatever the atomics make it: every row of a grouped product
 //   depends on that row alone, so the order changes no number).
@@ -21,6 +22,9 @@
 //   two accumulators (gate rows and up rows of the expert's stacked matrix), out = act(gate) * up in the operand
 //   type. Plain form: rows are the sorted rows themselves, out[pair] = weight[pair] * product in float, one row per
 //   pair, so that the sum over a token's pairs can be formed in a fixed order.
+//   `input_weight` (GLU form): both accumulators of a row times input_weight[pair] ahead of the activation, which is
+//   the expert applied to the weighted input (its products are linear). The plain form without a `pair_weight` leaves
+//   its rows unweighted.
 // mx_moe_combine: residual[t] += sum over the token's pairs, slot 0 first.
 // mx_moe_gather, mx_moe_combine_sorted: the ends of the tensor-core path. The grouped tcgen05 product
 //   (mx_gemm_tcgen05_grouped) reads its rows through TMA, so the tokens' rows are first copied into the order of
@@ -90,7 +94,7 @@ __device__ __forceinline__ void router_logits(const T* __restrict__ h, const flo
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const T* __restrict__ h, int ld, const float* __restrict__ router, int K, int n_experts, int top,
-                 int n_groups, int keep, float scale, int* __restrict__ ids, float* __restrict__ weights,
+                 int n_groups, int keep, float scale, int normalize, int* __restrict__ ids, float* __restrict__ weights,
                  int* __restrict__ counts, int* __restrict__ place) {
     extern __shared__ __align__(16) float route_s[];
     float* h_s = route_s;                         // [K]
@@ -121,6 +125,7 @@ moe_route_kernel(const T* __restrict__ h, int ld, const float* __restrict__ rout
             for (int g = lane; g < n_groups; g += 32)
                 if (worth[g] > v) { v = worth[g]; i = g; }
             arg_best(v, i);
+            if (i >= n_groups) i = 0;             // nothing comparable left (scores that are no numbers)
             __syncwarp();
             if (lane == 0) worth[i] = -3.f;
             for (int e = i * per + lane; e < (i + 1) * per; e += 32) open[e] = score[e];
@@ -135,6 +140,7 @@ moe_route_kernel(const T* __restrict__ h, int ld, const float* __restrict__ rout
         for (int e = lane; e < n_experts; e += 32)
             if (open[e] > v) { v = open[e]; i = e; }
         arg_best(v, i);
+        if (i >= n_experts) i = 0;                // nothing comparable left (scores that are no numbers)
         __syncwarp();
         if (lane == 0) open[i] = -3.f;
         __syncwarp();
@@ -146,7 +152,7 @@ moe_route_kernel(const T* __restrict__ h, int ld, const float* __restrict__ rout
             place[(size_t)t * top + slot] = atomicAdd(&counts[i], 1);
         }
     }
-    const float norm = scale / (total + 1e-20f);
+    const float norm = normalize ? scale / (total + 1e-20f) : scale;
     if (lane < min(top, 32)) {
         ids[(size_t)t * top + lane] = my_id;
         weights[(size_t)t * top + lane] = mine * norm;
@@ -266,7 +272,7 @@ __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ a, int lda, const int* __restrict__ order, int a_div, const T* __restrict__ w,
                 long long expert_stride, int N, int K, const int* __restrict__ tile_map,
                 const int* __restrict__ n_tiles, void* __restrict__ out_raw, const float* __restrict__ pair_weight,
-                const ClampedAct clamped) {
+                const ClampedAct clamped, const float* __restrict__ input_weight) {
     if ((int)blockIdx.y >= n_tiles[0]) return;
     __shared__ float a_s[MOE_BK][MOE_BM + 1], w_s[MOE_BK][MOE_BN + 1], u_s[GLU ? MOE_BK : 1][MOE_BN + 1];
     __shared__ int src_row[MOE_BM];
@@ -318,18 +324,19 @@ moe_gemm_kernel(const T* __restrict__ a, int lda, const int* __restrict__ order,
     for (int r = 0; r < 2; ++r) {
         const int row = 2 * ty + r;
         if (row >= rows) continue;
+        const float before = GLU && input_weight ? input_weight[order[row0 + row]] : 1.f;
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
             const int n = n0 + 4 * tx + c;
             if (n >= N) continue;
             if (GLU) {
-                const float g = acc[r][c];
-                const float value = ACT == 2 ? act_clamped(g, acc_u[r][c], clamped)
-                                             : (ACT == 0 ? gelu_tanh(g) : act_silu(g)) * acc_u[r][c];
+                const float g = acc[r][c] * before, u = acc_u[r][c] * before;
+                const float value = ACT == 2 ? act_clamped(g, u, clamped)
+                                             : (ACT == 0 ? gelu_tanh(g) : act_silu(g)) * u;
                 reinterpret_cast<T*>(out_raw)[(size_t)(row0 + row) * N + n] = from_float<T>(value);
             } else {
                 const int pair = order[row0 + row];
-                reinterpret_cast<float*>(out_raw)[(size_t)pair * N + n] = acc[r][c] * pair_weight[pair];
+                reinterpret_cast<float*>(out_raw)[(size_t)pair * N + n] = pair_weight ? acc[r][c] * pair_weight[pair] : acc[r][c];
             }
         }
     }
@@ -380,8 +387,9 @@ __global__ void moe_combine_sorted_kernel(const float* __restrict__ rows, const 
     for (int s = 0; s < top; ++s) {
         const long long pair = t * top + s;
         const int e = ids[pair];
-        if (e >= n_experts) sum += weight[pair] * to_float(input[(size_t)t * input_ld + c]);
-        else sum += weight[pair] * rows[((size_t)first[e] + place[pair]) * width + c];
+        const float w = weight ? weight[pair] : 1.f;
+        if (e >= n_experts) sum += w * to_float(input[(size_t)t * input_ld + c]);
+        else sum += w * rows[((size_t)first[e] + place[pair]) * width + c];
     }
     residual[i] += sum;
 }
@@ -408,7 +416,7 @@ __global__ void moe_combine_sorted_vec_kernel(const float* __restrict__ rows, co
     float4 sum = reinterpret_cast<const float4*>(residual)[i];
     for (int s = 0; s < top; ++s) {
         const long long pair = t * top + s;
-        const float w = weight[pair];
+        const float w = weight ? weight[pair] : 1.f;
         const int e = ids[pair];
         const float4 v = e >= n_experts ? load4(input + (size_t)t * input_ld + 4 * (size_t)c)
                                         : reinterpret_cast<const float4*>(rows)[((size_t)first[e] + place[pair]) * width4 + c];
@@ -418,19 +426,22 @@ __global__ void moe_combine_sorted_vec_kernel(const float* __restrict__ rows, co
 }
 
 template <typename T>
-__global__ void glu_kernel(const T* __restrict__ gu, int ld, T* __restrict__ out, int ff, int act, long long count) {
+__global__ void glu_kernel(const T* __restrict__ gu, int ld, T* __restrict__ out, int ff, int act, long long count,
+                           const float* __restrict__ pair_weight, const int* __restrict__ order) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= count) return;
     const long long t = i / ff;
     const int c = (int)(i - t * ff);
-    const float g = to_float(gu[(size_t)t * ld + c]);
-    const float u = to_float(gu[(size_t)t * ld + ff + c]);
+    const float before = pair_weight ? pair_weight[order[t]] : 1.f;
+    const float g = to_float(gu[(size_t)t * ld + c]) * before;
+    const float u = to_float(gu[(size_t)t * ld + ff + c]) * before;
     out[i] = from_float<T>((act == 0 ? gelu_tanh(g) : act_silu(g)) * u);
 }
 
 // eight neighbouring columns a thread, 16-byte accesses (bfloat16 rows whose width and stride are multiples of 8)
 __global__ void glu_vec_kernel(const __nv_bfloat16* __restrict__ gu, int ld, __nv_bfloat16* __restrict__ out, int ff,
-                               int act, long long groups) {
+                               int act, long long groups, const float* __restrict__ pair_weight,
+                               const int* __restrict__ order) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= groups) return;
     const int per_row = ff >> 3;
@@ -442,11 +453,12 @@ __global__ void glu_vec_kernel(const __nv_bfloat16* __restrict__ gu, int ld, __n
     const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uraw);
     uint4 oraw;
     __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&oraw);
+    const float before = pair_weight ? pair_weight[order[t]] : 1.f;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-        const float g0 = __low2float(g2[e]), g1 = __high2float(g2[e]);
+        const float g0 = __low2float(g2[e]) * before, g1 = __high2float(g2[e]) * before;
         const float a0 = act == 0 ? gelu_tanh(g0) : act_silu(g0), a1 = act == 0 ? gelu_tanh(g1) : act_silu(g1);
-        o2[e] = __floats2bfloat162_rn(a0 * __low2float(u2[e]), a1 * __high2float(u2[e]));
+        o2[e] = __floats2bfloat162_rn(a0 * (__low2float(u2[e]) * before), a1 * (__high2float(u2[e]) * before));
     }
     *reinterpret_cast<uint4*>(out + (size_t)t * ff + c) = oraw;
 }
@@ -454,8 +466,8 @@ __global__ void glu_vec_kernel(const __nv_bfloat16* __restrict__ gu, int ld, __n
 }  // namespace
 
 extern "C" int mx_moe_route(const void* h, int dtype, int ld, const float* router, int K, int n_experts, int top,
-                            int n_groups, int keep, float scale, int* ids, float* weights, int* counts, int* place,
-                            int n_tokens, cudaStream_t stream) {
+                            int n_groups, int keep, float scale, int normalize, int* ids, float* weights,
+                            int* counts, int* place, int n_tokens, cudaStream_t stream) {
     if (n_tokens <= 0) return MX_OK;
     if (n_experts <= 0 || top <= 0 || top > n_experts) MX_REFUSE("router: top %d of %d experts", top, n_experts);
     if (n_groups <= 0 || n_experts % n_groups != 0) MX_REFUSE("router: %d experts in %d equal groups", n_experts, n_groups);
@@ -465,10 +477,10 @@ extern "C" int mx_moe_route(const void* h, int dtype, int ld, const float* route
     if (smem > 48 * 1024) MX_REFUSE("router: %zu bytes of shared memory for K = %d and %d experts", smem, K, n_experts);
     if (dtype == MX_DTYPE_F32)
         moe_route_kernel<float><<<n_tokens, 256, smem, stream>>>((const float*)h, ld, router, K, n_experts, top, n_groups,
-                                                                keep, scale, ids, weights, counts, place);
+                                                                keep, scale, normalize, ids, weights, counts, place);
     else
         moe_route_kernel<__nv_bfloat16><<<n_tokens, 256, smem, stream>>>((const __nv_bfloat16*)h, ld, router, K, n_experts,
-                                                                        top, n_groups, keep, scale, ids, weights, counts,
+                                                                        top, n_groups, keep, scale, normalize, ids, weights, counts,
                                                                         place);
     return mx_launch_status();
 }
@@ -514,7 +526,7 @@ extern "C" int mx_moe_plan(const int* counts, const int* ids, const int* place, 
 extern "C" int mx_moe_gemm(const void* a, int dtype, int lda, const int* order, int a_div, const void* w,
                            long long expert_stride, int N, int K, const int* tile_map, const int* n_tiles, int max_tiles,
                            void* out, const float* pair_weight, int glu, int act, float limit, float slope, float shift,
-                           cudaStream_t stream) {
+                           const float* input_weight, cudaStream_t stream) {
     if (max_tiles <= 0 || N <= 0) return MX_OK;
     if (max_tiles > 65535) MX_REFUSE("routed feed-forward: %d row tiles exceed the grid", max_tiles);
     const dim3 grid((N + MOE_BN - 1) / MOE_BN, max_tiles);
@@ -522,7 +534,7 @@ extern "C" int mx_moe_gemm(const void* a, int dtype, int lda, const int* order, 
     if (glu && (act < 0 || act > 2)) MX_REFUSE("routed feed-forward: activation %d", act);
 #define MOE_LAUNCH(T, GLU, ACT)                                                                                        \
     moe_gemm_kernel<T, GLU, ACT><<<grid, 256, 0, stream>>>((const T*)a, lda, order, a_div, (const T*)w, expert_stride, \
-                                                           N, K, tile_map, n_tiles, out, pair_weight, clamped)
+                                                           N, K, tile_map, n_tiles, out, pair_weight, clamped, input_weight)
     if (dtype == MX_DTYPE_F32) {
         if (!glu) MOE_LAUNCH(float, false, 0);
         else if (act == 0) MOE_LAUNCH(float, true, 0);
@@ -596,20 +608,23 @@ extern "C" int mx_moe_combine(const float* pairs, float* residual, int n_tokens,
 }
 
 // out = act(gate) * up on rows [gate (ff) | up (ff)]; act 0 = gelu (tanh form), 1 = silu
-extern "C" int mx_glu(const void* gu, int ld, void* out, int dtype, int n_tokens, int ff, int act, cudaStream_t stream) {
+// `pair_weight` with `order` (sorted row -> pair; both or neither): gate and up of row r first times pair_weight[order[r]]
+extern "C" int mx_glu(const void* gu, int ld, void* out, int dtype, int n_tokens, int ff, int act,
+                      const float* pair_weight, const int* order, cudaStream_t stream) {
     const long long count = (long long)n_tokens * ff;
     if (count <= 0) return MX_OK;
     const unsigned blocks = (unsigned)((count + 255) / 256);
     if (dtype == MX_DTYPE_BF16 && ff % 8 == 0 && ld % 8 == 0 && ((uintptr_t)gu | (uintptr_t)out) % 16 == 0) {
         const long long groups = count >> 3;
         glu_vec_kernel<<<(unsigned)((groups + 255) / 256), 256, 0, stream>>>((const __nv_bfloat16*)gu, ld,
-                                                                             (__nv_bfloat16*)out, ff, act, groups);
+                                                                             (__nv_bfloat16*)out, ff, act, groups, pair_weight,
+                                                                             order);
         return mx_launch_status();
     }
     if (dtype == MX_DTYPE_F32)
-        glu_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gu, ld, (float*)out, ff, act, count);
+        glu_kernel<float><<<blocks, 256, 0, stream>>>((const float*)gu, ld, (float*)out, ff, act, count, pair_weight, order);
     else
         glu_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)gu, ld, (__nv_bfloat16*)out, ff, act,
-                                                             count);
+                                                             count, pair_weight, order);
     return mx_launch_status();
 }

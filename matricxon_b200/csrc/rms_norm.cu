@@ -2,6 +2,8 @@
 //
 //   unit(x) = x / sqrt(mean(x^2) + eps)          (eps inside the root)
 //   mx_rmsnorm:      out[r] = unit(x[rows ? rows[r] : r]) * (offset + weight)      (rows of x `x_stride` floats apart)
+//   mx_rmsnorm_pending: x[r] <- x[r] + acc[r] + col_bias (in place, float: the residual sum of a product whose float
+//                    accumulator acc is), then out[r] = unit(x[r]) * (offset + weight), in one pass
 //   mx_rmsnorm_branch_add: x[r] <- x[r] + unit(y[r]) * wb      (in place, float: a branch normalised on its way in)
 //                    out[r] <- unit(x[r]) * wn in the activation dtype (the next sublayer's normalised input;
 //                    wn null: x[r] itself, rounded; out null: nothing)
@@ -16,7 +18,8 @@
 // The float4 form of the post-norm sum takes part in chained launches (programmatic dependent launch).
 // One block per row; sums of squares are float and their order depends on the thread layout alone,
 // so a row's result does not depend on the other rows of the step.
-// mx_cast_rows rounds a float matrix to the activation dtype (the first sublayer's input).
+// mx_cast_rows rounds a float matrix to the activation dtype (the first sublayer's input); mx_cast_columns does the
+// same for a column range of wider rows.
 #include "common.cuh"
 
 namespace {
@@ -211,6 +214,52 @@ __global__ void rmsnorm_vec_kernel(const float* x, const int* __restrict__ rows,
     }
 }
 
+// The same behind a residual sum that is still to be formed: the row is x + (acc + col_bias), written back on the way.
+template <typename TOut>
+__global__ void rmsnorm_pending_vec_kernel(float* x, const float* acc, const float* __restrict__ col_bias,
+                                           const float* __restrict__ weight, float offset, TOut* __restrict__ out,
+                                           int hidden, float eps) {
+    __shared__ float scratch[32];
+    pdl_trigger();
+    const int r = blockIdx.x;
+    const int vecs = hidden >> 2;
+    float4 w[RMS_VEC];
+#pragma unroll
+    for (int n = 0; n < RMS_VEC; ++n) {                       // the weight does not depend on the kernel before
+        const int i = threadIdx.x + n * blockDim.x;
+        if (i < vecs) w[n] = reinterpret_cast<const float4*>(weight)[i];
+    }
+    pdl_wait();
+    float4* xr = reinterpret_cast<float4*>(after_wait(x) + (size_t)r * hidden);
+    const float4* ar = reinterpret_cast<const float4*>(after_wait(acc) + (size_t)r * hidden);
+    float4 kept[RMS_VEC];
+    float s = 0.f;
+#pragma unroll
+    for (int n = 0; n < RMS_VEC; ++n) {
+        const int i = threadIdx.x + n * blockDim.x;
+        if (i < vecs) {
+            const float4 a = xr[i];
+            float4 b = ar[i];
+            if (col_bias) {
+                const float4 c = reinterpret_cast<const float4*>(col_bias)[i];
+                b.x += c.x; b.y += c.y; b.z += c.z; b.w += c.w;
+            }
+            kept[n] = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+            xr[i] = kept[n];
+            s = fmaf(kept[n].x, kept[n].x, s); s = fmaf(kept[n].y, kept[n].y, s);
+            s = fmaf(kept[n].z, kept[n].z, s); s = fmaf(kept[n].w, kept[n].w, s);
+        }
+    }
+    const float inv = 1.0f / sqrtf(block_sum(s, scratch) / (float)hidden + eps);
+#pragma unroll
+    for (int n = 0; n < RMS_VEC; ++n) {
+        const int i = threadIdx.x + n * blockDim.x;
+        if (i < vecs)
+            store4(out + (size_t)r * hidden + 4 * i, kept[n].x * inv * (offset + w[n].x), kept[n].y * inv * (offset + w[n].y),
+                   kept[n].z * inv * (offset + w[n].z), kept[n].w * inv * (offset + w[n].w));
+    }
+}
+
 template <typename TAct>
 __global__ void rmsnorm_branch_add_vec_kernel(float* x, const float* y, const float* __restrict__ wb,
                                               const float* __restrict__ wn, TAct* out, int hidden, float eps) {
@@ -278,6 +327,14 @@ __global__ void cast_rows_kernel(const float* __restrict__ x, __nv_bfloat16* __r
     if (i < count) out[i] = __float2bfloat16_rn(x[i]);
 }
 
+__global__ void cast_columns_kernel(const float* __restrict__ x, int ld, __nv_bfloat16* __restrict__ out, int width,
+                                    long long count) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= count) return;
+    const long long r = i / width;
+    out[i] = __float2bfloat16_rn(x[(size_t)r * ld + (size_t)(i - r * width)]);
+}
+
 int threads_for(int hidden) { return hidden >= 4096 ? 512 : (hidden >= 1024 ? 256 : 128); }
 
 }  // namespace
@@ -303,6 +360,33 @@ extern "C" int mx_rmsnorm(const float* x, const int* rows, const float* weight, 
         rmsnorm_kernel<__nv_bfloat16><<<n_rows, threads, 0, stream>>>(x, rows, weight, offset,
                                                                      (__nv_bfloat16*)out, hidden, eps, x_stride);
     return mx_launch_status();
+}
+
+extern "C" int mx_epilogue(const void* acc, int acc_dtype, const float* bias, const float* residual, void* out,
+                           int out_dtype, long long n_rows, int n_cols, int mode, cudaStream_t stream);
+
+extern "C" int mx_rmsnorm_pending(float* x, const float* acc, const float* col_bias, const float* weight, float offset,
+                                  void* out, int out_dtype, int n_rows, int hidden, float eps, cudaStream_t stream) {
+    if (n_rows <= 0) return MX_OK;
+    if (hidden <= 0) MX_REFUSE("rmsnorm: hidden must be positive, got %d", hidden);
+    if (acc == nullptr) MX_REFUSE("rmsnorm of a pending sum: no accumulator");
+    const bool aligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(acc) |
+                           reinterpret_cast<uintptr_t>(col_bias) | reinterpret_cast<uintptr_t>(weight) |
+                           reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const int vec_threads = aligned ? vec_threads_for(n_rows, hidden) : 0;
+    if (vec_threads > 0) {
+        if (out_dtype == MX_DTYPE_F32)
+            mx_launch_chained(rmsnorm_pending_vec_kernel<float>, dim3(n_rows), dim3(vec_threads), 0, stream, x, acc,
+                              col_bias, weight, offset, (float*)out, hidden, eps);
+        else
+            mx_launch_chained(rmsnorm_pending_vec_kernel<__nv_bfloat16>, dim3(n_rows), dim3(vec_threads), 0, stream, x,
+                              acc, col_bias, weight, offset, (__nv_bfloat16*)out, hidden, eps);
+        return mx_launch_status();
+    }
+    // rows that the float4 kernel does not take: the sum by the epilogue kernel, then the norm
+    const int rc = mx_epilogue(acc, MX_DTYPE_F32, col_bias, x, x, MX_DTYPE_F32, n_rows, hidden, MX_MODE_RESIDUAL, stream);
+    if (rc != MX_OK) return rc;
+    return mx_rmsnorm(x, nullptr, weight, offset, out, out_dtype, n_rows, hidden, eps, hidden, stream);
 }
 
 extern "C" int mx_rmsnorm_branch_add(float* x, const float* y, const float* wb, const float* wn, void* out,
@@ -363,5 +447,12 @@ extern "C" int mx_rmsnorm_sum(float* x, const float* acc, float alpha, const flo
 extern "C" int mx_cast_rows(const float* x, void* out, long long count, cudaStream_t stream) {
     if (count <= 0) return MX_OK;
     cast_rows_kernel<<<(unsigned)((count + 255) / 256), 256, 0, stream>>>(x, (__nv_bfloat16*)out, count);
+    return mx_launch_status();
+}
+
+extern "C" int mx_cast_columns(const float* x, int ld, void* out, int n_rows, int width, cudaStream_t stream) {
+    const long long count = (long long)n_rows * width;
+    if (count <= 0) return MX_OK;
+    cast_columns_kernel<<<(unsigned)((count + 255) / 256), 256, 0, stream>>>(x, ld, (__nv_bfloat16*)out, width, count);
     return mx_launch_status();
 }

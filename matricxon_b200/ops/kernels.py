@@ -12,7 +12,7 @@ import torch
 from matricxon_b200.ops.library import KernelLibraryError, check, library
 
 F32, BF16 = 0, 1
-EPILOGUE_NONE, EPILOGUE_GELU, EPILOGUE_RESIDUAL, EPILOGUE_F32 = 0, 1, 2, 3
+EPILOGUE_NONE, EPILOGUE_GELU, EPILOGUE_RESIDUAL, EPILOGUE_F32, EPILOGUE_RELU2 = 0, 1, 2, 3, 4
 
 launch_count = 0      # kernels of this library launched so far in this process
 
@@ -368,6 +368,14 @@ def _sink_ptr(sink: torch.Tensor | None, n_heads: int) -> int | None:
     return sink.data_ptr()
 
 
+def _distance_ptr(distance: torch.Tensor | None, n_heads: int) -> int | None:
+    if distance is None:
+        return None
+    _need(distance, "distance", torch.float32)
+    assert tuple(distance.shape) == (2, n_heads), (distance.shape, n_heads)
+    return distance.data_ptr()
+
+
 def attention_scratch_bytes(n_tokens: int, n_heads: int, head_dim: int, n_splits: int) -> int:
     return int(library().mx_attention_scratch_bytes(n_tokens, n_heads, head_dim, n_splits))
 
@@ -377,25 +385,27 @@ def paged_attention(q: torch.Tensor, q_stride: int, cache: torch.Tensor, block_t
                     n_kv_heads: int, head_dim: int, window: int | None, scale: float,
                     out: torch.Tensor, status: torch.Tensor, n_splits: int = 1,
                     scratch: torch.Tensor | None = None, softcap: float | None = None,
-                    sink: torch.Tensor | None = None, keep_first: int = 0) -> None:
+                    sink: torch.Tensor | None = None, keep_first: int = 0,
+                    distance: torch.Tensor | None = None) -> None:
     """Attention of ``n_tokens`` query rows over the paged cache.
 
     ``q`` points at the first query head of row 0 and rows are ``q_stride`` elements apart
     (so the q part of a fused qkv buffer can be used in place). ``out`` is [tokens, heads * dim].
     ``softcap``: scaled scores become ``softcap * tanh(score / softcap)``. ``sink`` (float32, one per
     head): ``exp(sink[h])`` joins the softmax's denominator and brings no value. ``keep_first``: with a
-    window, the keys at positions below it stay visible at any distance.
+    window, the keys at positions below it stay visible at any distance. ``distance`` (float32 [2, heads], rows r1 and
+    r2): the (capped) score of the query at p and the key at j loses ``r1 ln(1 + r2 (p - j))``.
     """
     _need(q, "q", contiguous=False)
     _need(cache, "cache", q.dtype)
     _need(block_tables, "block_tables", torch.int32)
     _need(tok_seq, "tok_seq", torch.int32)
     _need(positions, "positions", torch.int32)
-    _need(out, "out", q.dtype)
+    _need(out, "out", q.dtype, contiguous=False)
     _need(status, "status", torch.int32)
     page_size = cache.shape[3]
     assert tuple(cache.shape[1:]) == (2, n_kv_heads, page_size, head_dim), cache.shape
-    assert out.shape[1] == n_heads * head_dim and out.shape[0] >= n_tokens
+    assert out.shape[1] == n_heads * head_dim and out.shape[0] >= n_tokens and out.stride(1) == 1
     if n_splits > 1:
         need = attention_scratch_bytes(n_tokens, n_heads, head_dim, n_splits)
         if scratch is None or scratch.numel() * scratch.element_size() < need:
@@ -406,7 +416,7 @@ def paged_attention(q: torch.Tensor, q_stride: int, cache: torch.Tensor, block_t
         _ptr(block_tables), block_tables.stride(0), _ptr(tok_seq), _ptr(positions), n_tokens,
         n_heads, n_kv_heads, head_dim, int(window or 0), float(scale), _ptr(out), out.stride(0),
         n_splits, _ptr(scratch), _ptr(status), float(softcap or 0.0), _sink_ptr(sink, n_heads), int(keep_first),
-        _stream()), "paged_attention")
+        _distance_ptr(distance, n_heads), _stream()), "paged_attention")
     _launched(2 if n_splits > 1 else 1)
 
 
@@ -448,7 +458,8 @@ def paged_attention_tc(q: torch.Tensor, q_stride: int, cache: torch.Tensor, bloc
                        n_tokens: int, n_heads: int, n_kv_heads: int, head_dim: int, window: int | None,
                        scale: float, out: torch.Tensor, status: torch.Tensor, n_splits: int = 1,
                        scratch: torch.Tensor | None = None, softcap: float | None = None,
-                       sink: torch.Tensor | None = None, keep_first: int = 0) -> None:
+                       sink: torch.Tensor | None = None, keep_first: int = 0,
+                    distance: torch.Tensor | None = None) -> None:
     """Attention of prompt portions on tcgen05 (bfloat16, head_dim 128, pages of 16 or 32). Under a window the
     sequence's first ``keep_first`` keys stay visible.
     ``tiles`` is int32 [n_tiles, 2]: (sequence, first token) of tiles of 128 // group tokens
@@ -460,10 +471,10 @@ def paged_attention_tc(q: torch.Tensor, q_stride: int, cache: torch.Tensor, bloc
     for name, tensor in (("block_tables", block_tables), ("cu_q", cu_q),
                          ("context_lens", context_lens), ("tiles", tiles), ("status", status)):
         _need(tensor, name, torch.int32)
-    _need(out, "out", torch.bfloat16)
+    _need(out, "out", torch.bfloat16, contiguous=False)
     page_size = cache.shape[3]
     assert tuple(cache.shape[1:]) == (2, n_kv_heads, page_size, head_dim), cache.shape
-    assert out.shape[1] == n_heads * head_dim and out.shape[0] >= n_tokens and q.shape[0] >= n_tokens
+    assert out.shape[1] == n_heads * head_dim and out.shape[0] >= n_tokens and out.stride(1) == 1 and q.shape[0] >= n_tokens
     assert tiles.numel() >= 2 * n_tiles
     if n_splits > 1:
         _need(scratch, "scratch", torch.float32)
@@ -473,7 +484,8 @@ def paged_attention_tc(q: torch.Tensor, q_stride: int, cache: torch.Tensor, bloc
         block_tables.stride(0), _ptr(cu_q), _ptr(context_lens), _ptr(tiles), n_tiles, n_tokens,
         n_heads, n_kv_heads, head_dim, int(window or 0), float(scale), _ptr(out), out.stride(0),
         int(n_splits), _ptr(scratch) if n_splits > 1 else None, _ptr(status), float(softcap or 0.0),
-        _sink_ptr(sink, n_heads), int(keep_first) if window else 0, _stream()), "paged_attention_tc")
+        _sink_ptr(sink, n_heads), int(keep_first) if window else 0, _distance_ptr(distance, n_heads), _stream()),
+        "paged_attention_tc")
     _launched()
 
 
@@ -483,7 +495,8 @@ def paged_attention_mma(q: torch.Tensor, q_stride: int, cache: torch.Tensor,
                         n_kv_heads: int, head_dim: int, window: int | None, scale: float,
                         out: torch.Tensor, status: torch.Tensor, n_splits: int = 1,
                         scratch: torch.Tensor | None = None, softcap: float | None = None,
-                        sink: torch.Tensor | None = None, keep_first: int = 0) -> None:
+                        sink: torch.Tensor | None = None, keep_first: int = 0,
+                    distance: torch.Tensor | None = None) -> None:
     """Tensor-core attention (bfloat16, head_dim 64 or 128). ``tiles`` is int32 [n_tiles, 2]:
     (sequence, first row) of each tile of the (token, head-in-group) rows; ``narrow`` tiles
     hold at most 16 rows, the others 64 (see ``attention_tile_lists``)."""
@@ -492,10 +505,10 @@ def paged_attention_mma(q: torch.Tensor, q_stride: int, cache: torch.Tensor,
     for name, tensor in (("block_tables", block_tables), ("cu_q", cu_q),
                          ("context_lens", context_lens), ("status", status)):
         _need(tensor, name, torch.int32)
-    _need(out, "out", torch.bfloat16)
+    _need(out, "out", torch.bfloat16, contiguous=False)
     page_size = cache.shape[3]
     assert tuple(cache.shape[1:]) == (2, n_kv_heads, page_size, head_dim), cache.shape
-    assert out.shape[1] == n_heads * head_dim and out.shape[0] >= n_tokens
+    assert out.shape[1] == n_heads * head_dim and out.shape[0] >= n_tokens and out.stride(1) == 1
     if tiles is None:
         # no list: tile i is the whole of sequence i (narrow tiles only: every sequence brings at most 16 rows)
         assert narrow and n_tiles <= context_lens.numel()
@@ -512,7 +525,7 @@ def paged_attention_mma(q: torch.Tensor, q_stride: int, cache: torch.Tensor,
         block_tables.stride(0), _ptr(cu_q), _ptr(context_lens), _ptr(tiles) if tiles is not None else None, n_tiles,
         1 if narrow else 0, n_tokens, n_heads, n_kv_heads, head_dim, int(window or 0), float(scale),
         _ptr(out), out.stride(0), n_splits, _ptr(scratch), _ptr(status), float(softcap or 0.0),
-        _sink_ptr(sink, n_heads), int(keep_first), _stream()), "paged_attention_mma")
+        _sink_ptr(sink, n_heads), int(keep_first), _distance_ptr(distance, n_heads), _stream()), "paged_attention_mma")
     _launched(2 if n_splits > 1 else 1)
 
 
@@ -554,6 +567,24 @@ def rmsnorm_sum(x: torch.Tensor, acc: torch.Tensor, alpha: float, weight: torch.
     check(library().mx_rmsnorm_sum(_ptr(x), _ptr(acc), float(alpha), _ptr(weight), float(offset), _ptr(act),
                                    dtype_code(act.dtype) if act is not None else F32, x.shape[0], x.shape[1],
                                    float(eps), _stream()), "rmsnorm_sum")
+    _launched()
+
+
+def rmsnorm_pending(x: torch.Tensor, acc: torch.Tensor, col_bias: torch.Tensor | None, weight: torch.Tensor,
+                    offset: float, eps: float, out: torch.Tensor) -> None:
+    """``x += acc + col_bias`` (the residual epilogue of a product whose float accumulator is ``acc``), then
+    ``out = x / sqrt(mean(x^2) + eps) * (offset + weight)``, in one pass over the rows."""
+    _need(x, "x", torch.float32)
+    _need(acc, "acc", torch.float32)
+    _need(weight, "weight", torch.float32)
+    _need(out, "out")
+    assert acc.shape == x.shape and out.shape == x.shape and weight.numel() == x.shape[1]
+    if col_bias is not None:
+        _need(col_bias, "col_bias", torch.float32)
+        assert col_bias.numel() == x.shape[1]
+    check(library().mx_rmsnorm_pending(_ptr(x), _ptr(acc), _ptr(col_bias), _ptr(weight), float(offset), _ptr(out),
+                                       dtype_code(out.dtype), x.shape[0], x.shape[1], float(eps), _stream()),
+          "rmsnorm_pending")
     _launched()
 
 
@@ -1011,17 +1042,19 @@ def gla_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, decay: torc
     _launched()
 
 
-def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor,
                   n_heads: int, vdim: int) -> None:
     """out[t, h, e] = unit(o[t, h])[e] * weight[e] * silu(gate[t, h, e]); unit is the RMS norm over one head's
-    ``vdim`` entries with eps inside the root; ``gate`` a float32 view with any row stride."""
+    ``vdim`` entries with eps inside the root; ``weight`` None: no weight; ``gate`` a float32 view with any row stride."""
     _need(o, "o", torch.float32)
     _need(gate, "gate", torch.float32, contiguous=False)
-    _need(weight, "weight", torch.float32)
+    if weight is not None:
+        _need(weight, "weight", torch.float32)
+        assert weight.numel() == vdim
     _need(out, "out")
     n = o.shape[0]
     assert tuple(o.shape) == (n, n_heads * vdim) and tuple(gate.shape) == (n, n_heads * vdim) and gate.stride(1) == 1
-    assert tuple(out.shape) == (n, n_heads * vdim) and weight.numel() == vdim
+    assert tuple(out.shape) == (n, n_heads * vdim)
     check(library().mx_gla_norm_gate(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), float(eps), _ptr(out),
                                      dtype_code(out.dtype), n, n_heads, vdim, _stream()), "gla_norm_gate")
     _launched()
@@ -1032,14 +1065,21 @@ GLU_ACTIVATIONS = {"gelu_tanh": 0, "silu": 1}
 CLAMPED_ACTIVATION = 2       # the grouped product's code for ``min(g, limit) * sigmoid(slope g) * (clamp(u) + shift)``
 
 
-def glu(gate_up: torch.Tensor, out: torch.Tensor, activation: str) -> None:
-    """Rows ``[gate | up]`` -> ``act(gate) * up``."""
+def glu(gate_up: torch.Tensor, out: torch.Tensor, activation: str, pair_weight: torch.Tensor | None = None,
+        order: torch.Tensor | None = None) -> None:
+    """Rows ``[gate | up]`` -> ``act(gate) * up``; with ``pair_weight`` (float32 per pair) and ``order`` (int32, the
+    pair of every row) both halves of row r are multiplied by ``pair_weight[order[r]]`` first."""
+    if pair_weight is not None:
+        _need(pair_weight, "pair_weight", torch.float32)
+        _need(order, "order", torch.int32)
+        assert order.numel() == gate_up.shape[0] == pair_weight.numel()
     _need(gate_up, "gate_up")
     _need(out, "out", gate_up.dtype)
     n, ff = out.shape
     assert tuple(gate_up.shape) == (n, 2 * ff)
     check(library().mx_glu(_ptr(gate_up), gate_up.stride(0), _ptr(out), dtype_code(out.dtype), n, ff,
-                           GLU_ACTIVATIONS[activation], _stream()), "glu")
+                           GLU_ACTIVATIONS[activation], _ptr(pair_weight), _ptr(order) if pair_weight is not None else None,
+                           _stream()), "glu")
     _launched()
 
 
@@ -1048,9 +1088,11 @@ def moe_tile_rows() -> int:
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, n_groups: int, keep: int, scale: float,
-              ids: torch.Tensor, weights: torch.Tensor, counts: torch.Tensor, place: torch.Tensor) -> None:
+              ids: torch.Tensor, weights: torch.Tensor, counts: torch.Tensor, place: torch.Tensor,
+              normalize: bool = True) -> None:
     """Per token: sigmoid scores of the float32 router [experts, K], the ``top`` best experts of the ``keep`` best
-    of ``n_groups`` runs of neighbours (a run is worth its two best scores), weights = scores / their sum * scale.
+    of ``n_groups`` runs of neighbours (a run is worth its two best scores), weights = scores / their sum * scale
+    (not ``normalize``: scores * scale).
     ``counts`` [experts] must be zero; afterwards it holds every expert's pairs and ``place`` each pair's index
     among them."""
     _need(h, "h")
@@ -1063,8 +1105,8 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, top: int, n_groups: int, ke
     assert router.shape[1] == k and ids.numel() == n * top == weights.numel() == place.numel()
     assert counts.numel() == n_experts
     check(library().mx_moe_route(_ptr(h), dtype_code(h.dtype), h.stride(0), _ptr(router), k, n_experts, top, n_groups,
-                                 keep, float(scale), _ptr(ids), _ptr(weights), _ptr(counts), _ptr(place), n, _stream()),
-          "moe_route")
+                                 keep, float(scale), 1 if normalize else 0, _ptr(ids), _ptr(weights), _ptr(counts), _ptr(place), n,
+                                 _stream()), "moe_route")
     _launched()
 
 
@@ -1093,11 +1135,12 @@ def moe_max_tiles(n_pairs: int, n_experts: int, tile_rows: int | None = None) ->
 
 def moe_gemm(a: torch.Tensor, order: torch.Tensor, a_div: int, w: torch.Tensor, tile_map: torch.Tensor,
              n_tiles: torch.Tensor, max_tiles: int, out: torch.Tensor, pair_weight: torch.Tensor | None,
-             activation: str | tuple | None) -> None:
+             activation: str | tuple | None, input_weight: torch.Tensor | None = None) -> None:
     """The grouped product over the pairs sorted by expert. With ``activation``: ``a`` holds the tokens' rows (pair
     p reads row ``p // a_div``), ``w`` [experts, 2 N, K] stacks gate and up rows, ``out`` [pairs, N] (sorted order,
     dtype of a) = act(gate) * up. Without: ``a`` [pairs, K] is in sorted order, ``w`` [experts, N, K], ``out``
-    float32 [pairs, N] in pair order = ``pair_weight[pair] *`` product. ``activation`` is a name of
+    float32 [pairs, N] in pair order = ``pair_weight[pair] *`` product (None: the product). ``input_weight`` (float32
+    per pair, with an activation): the pair's row counts as ``input_weight[pair] * row``. ``activation`` is a name of
     ``GLU_ACTIVATIONS`` or ``("clamped", limit, slope, shift)``: ``g = min(gate, limit)``,
     ``u = clamp(up, -limit, limit)`` (limit <= 0: neither), ``g * sigmoid(slope g) * (u + shift)``."""
     _need(a, "a")
@@ -1112,8 +1155,11 @@ def moe_gemm(a: torch.Tensor, order: torch.Tensor, a_div: int, w: torch.Tensor, 
     if glu_form:
         assert out.dtype == a.dtype
     else:
-        _need(pair_weight, "pair_weight", torch.float32)
         assert out.dtype == torch.float32
+    for name, weight in (("pair_weight", pair_weight), ("input_weight", input_weight)):
+        if weight is not None:
+            _need(weight, name, torch.float32)
+            assert weight.numel() == order.numel()
     code, constants = 0, (0.0, 0.0, 0.0)
     if isinstance(activation, tuple):
         code, constants = CLAMPED_ACTIVATION, tuple(float(c) for c in activation[1:4])
@@ -1121,7 +1167,7 @@ def moe_gemm(a: torch.Tensor, order: torch.Tensor, a_div: int, w: torch.Tensor, 
         code = GLU_ACTIVATIONS[activation]
     check(library().mx_moe_gemm(_ptr(a), dtype_code(a.dtype), a.stride(0), _ptr(order), a_div, _ptr(w), w.stride(0), n, k,
                                 _ptr(tile_map), _ptr(n_tiles), max_tiles, _ptr(out), _ptr(pair_weight),
-                                1 if glu_form else 0, code, *constants, _stream()),
+                                1 if glu_form else 0, code, *constants, _ptr(input_weight), _stream()),
           "moe_gemm")
     _launched()
 
@@ -1230,17 +1276,19 @@ def gemm_tcgen05_grouped(a: torch.Tensor, w: torch.Tensor, tile_map: torch.Tenso
 
 
 def moe_combine_sorted(rows: torch.Tensor, ids: torch.Tensor, place: torch.Tensor, first: torch.Tensor,
-                       weights: torch.Tensor, residual: torch.Tensor, top: int, identity=None) -> None:
+                       weights: torch.Tensor | None, residual: torch.Tensor, top: int, identity=None) -> None:
     """residual[t] += sum over the token's ``top`` pairs of ``weights[pair] * rows[first[ids[pair]] + place[pair]]``
-    (``rows`` float32 [pairs, width] in sorted order), first slot first. ``identity`` = (input [tokens, width],
+    (``rows`` float32 [pairs, width] in sorted order; ``weights`` None: every weight is one), first slot first. ``identity`` = (input [tokens, width],
     n_experts): a pair whose id is ``>= n_experts`` has no row; its token's input stands for it."""
     _need(rows, "rows", torch.float32)
     _need(residual, "residual", torch.float32)
-    _need(weights, "weights", torch.float32)
+    if weights is not None:
+        _need(weights, "weights", torch.float32)
+        assert weights.numel() == ids.numel()
     for name, tensor in (("ids", ids), ("place", place), ("first", first)):
         _need(tensor, name, torch.int32)
     n, width = residual.shape
-    assert tuple(rows.shape) == (n * top, width) and ids.numel() == n * top == place.numel() == weights.numel()
+    assert tuple(rows.shape) == (n * top, width) and ids.numel() == n * top == place.numel()
     _, _, source, code, ld, n_experts = _identity_arguments(
         None if identity is None else (ids, weights, identity[0], identity[1]), n, width)
     check(library().mx_moe_combine_sorted(_ptr(rows), _ptr(ids), _ptr(place), _ptr(first), _ptr(weights), _ptr(residual),
@@ -1357,13 +1405,15 @@ def rotate_norm_kv_write(proj: torch.Tensor, positions: torch.Tensor, freq: torc
 def norm_rotate_kv_write(proj: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, rot: int, interleaved: bool,
                          q_weight: torch.Tensor | None, k_weight: torch.Tensor | None, eps: float,
                          slots: torch.Tensor | None, cache: torch.Tensor | None, q_out: torch.Tensor, n_heads: int,
-                         n_kv_heads: int, dim: int, vdim: int, status: torch.Tensor) -> None:
+                         n_kv_heads: int, dim: int, vdim: int, status: torch.Tensor, amplitude: float = 1.0,
+                         values_are_keys: bool = False, value_scale: float = 1.0) -> None:
     """From float rows ``[q | k | v | ...]`` of a fused projection: q and k heads RMS-normalised over ``dim`` with the
     weights ``q_weight`` / ``k_weight`` (float32 [dim]; None: left as they are; ``eps`` inside the root) and then
     rotated over their first ``rot`` entries (pairs (i, i + rot/2) or, ``interleaved``, (2i, 2i + 1); angle
-    ``position * freq[i]``); q into ``q_out`` [tokens, heads * hd], k and v into the paged ``cache``
-    [pages, 2, kv heads, page_size, hd] at ``slots`` (both None: nothing is stored). ``hd`` is the padded head size of
-    ``q_out``; tails are zero."""
+    ``position * freq[i]``, cos and sin times ``amplitude``); q into ``q_out`` [tokens, heads * hd], k and v into the
+    paged ``cache`` [pages, 2, kv heads, page_size, hd] at ``slots`` (both None: nothing is stored). ``hd`` is the padded
+    head size of ``q_out``; tails are zero. Values are stored times ``value_scale``; ``values_are_keys``: they are the
+    keys as projected, before norm and rotation, and the rows hold no v."""
     _need(proj, "proj", torch.float32, contiguous=False)
     _need(positions, "positions", torch.int32)
     _need(freq, "freq", torch.float32)
@@ -1384,8 +1434,193 @@ def norm_rotate_kv_write(proj: torch.Tensor, positions: torch.Tensor, freq: torc
         n_pages, page_size = cache.shape[0], cache.shape[3]
         assert tuple(cache.shape[1:]) == (2, n_kv_heads, page_size, hd), cache.shape
     check(library().mx_norm_rotate_kv_write(_ptr(proj), proj.stride(0), _ptr(positions), _ptr(freq), int(rot),
-                                            1 if interleaved else 0, _ptr(q_weight), _ptr(k_weight), float(eps),
-                                            _ptr(slots) if cache is not None else None, _ptr(cache), n_pages, page_size,
+                                            1 if interleaved else 0, float(amplitude), _ptr(q_weight), _ptr(k_weight),
+                                            float(eps), _ptr(slots) if cache is not None else None, _ptr(cache), n_pages, page_size,
                                             _ptr(q_out), dtype_code(q_out.dtype), n, n_heads, n_kv_heads, dim, vdim, hd,
-                                            _ptr(status), _stream()), "norm_rotate_kv_write")
+                                            1 if values_are_keys else 0, float(value_scale), _ptr(status), _stream()),
+          "norm_rotate_kv_write")
+    _launched()
+
+
+# ---------------------------------------------------------------------- retention
+def rotate_heads(rows: torch.Tensor, col: int, n_heads: int, dim: int, rot: int, positions: torch.Tensor,
+                 freq: torch.Tensor) -> None:
+    """The first ``rot`` entries of ``n_heads`` heads of ``dim`` entries, side by side from column ``col`` of float
+    rows, rotated in place (pairs (i, i + rot/2), angle ``position * freq[i]``)."""
+    _need(rows, "rows", torch.float32, contiguous=False)
+    _need(positions, "positions", torch.int32)
+    _need(freq, "freq", torch.float32)
+    n = rows.shape[0]
+    assert rows.stride(1) == 1 and rows.shape[1] >= col + n_heads * dim and freq.numel() >= rot // 2
+    assert positions.numel() >= n
+    check(library().mx_rotate_heads(_ptr(rows), rows.stride(0), int(col), n, n_heads, dim, int(rot), _ptr(positions),
+                                    _ptr(freq), _stream()), "rotate_heads")
+    _launched()
+
+
+def retention_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, head_decay: torch.Tensor, q_scale: float,
+                   state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor,
+                   n_heads: int, dim: int, vdim: int, positions: torch.Tensor | None = None,
+                   freq: torch.Tensor | None = None, rot: int = 0) -> None:
+    """``S <- head_decay_h S + k_t v_t^T; out_t = S^T (q_scale * q_t)`` over every sequence's tokens in order, from and
+    to ``state`` [slots, heads, dim, vdim] (float32); q, k and v are column ranges of the float rows ``proj``. With
+    ``freq`` q and k are rotated over their first ``rot`` entries on their way in."""
+    for name, tensor in (("proj", proj), ("head_decay", head_decay), ("state", state), ("out", out)):
+        _need(tensor, name, torch.float32)
+    n = proj.shape[0]
+    assert tuple(state.shape[1:]) == (n_heads, dim, vdim), state.shape
+    assert head_decay.numel() == n_heads and tuple(out.shape) == (n, n_heads * vdim)
+    if freq is not None:
+        _need(freq, "freq", torch.float32)
+        _need(positions, "positions", torch.int32)
+        assert freq.numel() >= rot // 2 and positions.numel() >= n
+    check(library().mx_retention_scan(_ptr(proj), proj.stride(0), q_col, k_col, v_col, _ptr(head_decay), float(q_scale),
+                                      _ptr(state), _ptr(cu_q), _ptr(state_slots), _ptr(out), n_seqs, n_heads, dim, vdim,
+                                      _ptr(positions) if freq is not None else None, _ptr(freq), int(rot), _stream()),
+          "retention_scan")
+    _launched()
+
+
+# ---------------------------------------------------------------------- short convolutions, selective recurrence
+def conv_norm_kv_write(proj: torch.Tensor, bias: torch.Tensor | None, conv: torch.Tensor, q_weight: torch.Tensor,
+                       k_weight: torch.Tensor | None, eps: float, temperature: tuple[float, float], state: torch.Tensor | None,
+                       positions: torch.Tensor, tok_seq: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor,
+                       slots: torch.Tensor | None, cache: torch.Tensor | None, q_out: torch.Tensor, n_heads: int,
+                       n_kv_heads: int, dim: int, vdim: int, status: torch.Tensor) -> None:
+    """From float rows ``[q | k | v]`` of a fused projection (``k_weight`` None: rows of q alone): plus ``bias``, through
+    a causal convolution per channel (``conv`` float32 [taps, channels], continuing from ``state`` [slots, >= (taps - 1) *
+    channels]), q and k divided by their root mean square over ALL their channels times their weights, q times
+    ``1 + coef ln(floor((position + 1) / every) + 1)`` (``temperature`` = (coef, every)); q into ``q_out``
+    [tokens, heads * hd], k and v into the pages at ``slots``, heads padded with zeros to hd. The state of sequences that
+    bring one token is moved on here, that of the others by ``conv_state_update`` afterwards."""
+    for name, tensor in (("proj", proj), ("conv", conv), ("q_weight", q_weight)):
+        _need(tensor, name, torch.float32, contiguous=name != "proj")
+    if state is None:
+        assert conv.shape[0] == 1, "a convolution of two or more taps keeps its latest inputs"
+    else:
+        _need(state, "state", torch.float32)
+    for name, tensor in (("positions", positions), ("tok_seq", tok_seq), ("cu_q", cu_q), ("state_slots", state_slots),
+                         ("status", status)):
+        _need(tensor, name, torch.int32)
+    _need(q_out, "q_out")
+    n = q_out.shape[0]
+    hd = q_out.shape[1] // n_heads
+    own = k_weight is not None
+    channels = n_heads * dim + (n_kv_heads * (dim + vdim) if own else 0)
+    assert q_out.shape[1] == n_heads * hd and proj.stride(1) == 1 and proj.shape[0] >= n and proj.shape[1] >= channels
+    assert conv.shape[1] == channels and q_weight.numel() == n_heads * dim
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        assert bias.numel() == channels
+    n_pages, page_size = 0, 1
+    if own:
+        _need(k_weight, "k_weight", torch.float32)
+        assert k_weight.numel() == n_kv_heads * dim
+    if cache is not None:
+        _need(cache, "cache", q_out.dtype)
+        _need(slots, "slots", torch.int32)
+        n_pages, page_size = cache.shape[0], cache.shape[3]
+        assert tuple(cache.shape[1:]) == (2, n_kv_heads, page_size, hd), cache.shape
+    coef, every = temperature
+    check(library().mx_conv_norm_kv_write(
+        _ptr(proj), proj.stride(0), _ptr(bias), _ptr(conv), conv.shape[0], _ptr(q_weight), _ptr(k_weight), float(eps),
+        float(coef), float(every), _ptr(state), state.stride(0) if state is not None else 0, _ptr(positions), _ptr(tok_seq), _ptr(cu_q),
+        _ptr(state_slots), _ptr(slots) if cache is not None else None, _ptr(cache), n_pages, page_size, _ptr(q_out),
+        dtype_code(q_out.dtype), n, n_heads, n_kv_heads, dim, vdim, hd, 1 if own else 0, _ptr(status), _stream()),
+        "conv_norm_kv_write")
+    _launched()
+
+
+def conv_state_update(rows: torch.Tensor, bias: torch.Tensor | None, state: torch.Tensor, cu_q: torch.Tensor,
+                      state_slots: torch.Tensor, n_seqs: int, channels: int, taps: int) -> None:
+    """Leaves the latest ``taps - 1`` convolution inputs (``rows`` [tokens, >= channels] plus ``bias``) of every sequence
+    that brings two or more tokens at the start of its ``state`` vector."""
+    _need(rows, "rows", contiguous=False)
+    _need(state, "state", torch.float32)
+    assert rows.stride(1) == 1 and rows.shape[1] >= channels and state.stride(0) >= (taps - 1) * channels
+    if bias is not None:
+        _need(bias, "bias", torch.float32)
+        assert bias.numel() == channels
+    check(library().mx_conv_state_update(_ptr(rows), dtype_code(rows.dtype), rows.stride(0), _ptr(bias), _ptr(state),
+                                         state.stride(0), _ptr(cu_q), _ptr(state_slots), n_seqs, channels, taps,
+                                         _stream()), "conv_state_update")
+    _launched()
+
+
+def conv_silu(x: torch.Tensor, conv: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, tok_seq: torch.Tensor,
+              cu_q: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor) -> None:
+    """out = silu(causal convolution of ``x`` + ``bias``) per channel; ``x`` [tokens, channels] may be a column range of
+    wider rows (float32 or the dtype of ``out``), ``conv`` is float32 [taps, channels], the earlier inputs come from the
+    start of ``state`` [slots, ...]. State rules as in ``conv_norm_kv_write``."""
+    _need(x, "x", contiguous=False)
+    _need(conv, "conv", torch.float32)
+    _need(bias, "bias", torch.float32)
+    _need(state, "state", torch.float32)          # every slot's vector; with one tap nothing of it is convolution inputs
+    _need(out, "out")
+    n, channels = out.shape
+    taps = conv.shape[0]
+    assert x.stride(1) == 1 and tuple(x.shape) == (n, channels) and conv.shape[1] == channels == bias.numel()
+    check(library().mx_conv_silu(_ptr(x), dtype_code(x.dtype), x.stride(0), _ptr(conv), _ptr(bias), _ptr(state),
+                                 state.stride(0), _ptr(tok_seq), _ptr(cu_q), _ptr(state_slots), _ptr(out),
+                                 dtype_code(out.dtype), n, channels, taps, _stream()), "conv_silu")
+    _launched()
+
+
+def _scan_operands(u, low, dt_bias, a_log2, d, z, state, state_offset, out, n_states, dt_rank):
+    _need(u, "u")
+    _need(low, "low", torch.float32)
+    for name, tensor in (("dt_bias", dt_bias), ("a_log2", a_log2), ("d", d), ("state", state)):
+        _need(tensor, name, torch.float32)
+    _need(z, "z", contiguous=False)
+    _need(out, "out", u.dtype, contiguous=False)
+    n, channels = u.shape
+    assert tuple(a_log2.shape) == (channels, n_states) and dt_bias.numel() == channels == d.numel()
+    assert tuple(z.shape) == (n, channels) and z.stride(1) == 1 and tuple(out.shape) == (n, channels) and out.stride(1) == 1
+    assert low.shape[1] >= dt_rank + 2 * n_states and state.stride(0) >= state_offset + channels * n_states
+    return n, channels
+
+
+def selective_scan(u: torch.Tensor, raw: torch.Tensor, low: torch.Tensor, dt_bias: torch.Tensor, a_log2: torch.Tensor,
+                   d: torch.Tensor, z: torch.Tensor, state: torch.Tensor, state_offset: int, cu_q: torch.Tensor,
+                   state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor, n_states: int, dt_rank: int,
+                   out_scale: float = 1.0) -> None:
+    """Every sequence's tokens in order, from and to the recurrent part of its ``state`` vector ([channels, n_states] at
+    ``state_offset``): ``dt = softplus(raw + dt_bias)``, ``S <- exp(dt A) S + dt u B``,
+    ``out = (S C + d u) * silu(z) * out_scale``. ``raw`` float32 [tokens, channels]; ``low`` float32 rows
+    ``[dt_rank | B | C]``; ``a_log2`` is A * log2(e); ``u`` and ``out`` in the activation dtype, ``z`` in it or float32."""
+    n, channels = _scan_operands(u, low, dt_bias, a_log2, d, z, state, state_offset, out, n_states, dt_rank)
+    _need(raw, "raw", torch.float32)
+    assert tuple(raw.shape) == (n, channels)
+    check(library().mx_selective_scan(_ptr(u), _ptr(raw), raw.stride(0), _ptr(low), low.stride(0), _ptr(dt_bias),
+                                      _ptr(a_log2), _ptr(d), _ptr(z), dtype_code(z.dtype), z.stride(0), _ptr(state),
+                                      state.stride(0), int(state_offset), _ptr(cu_q), _ptr(state_slots), _ptr(out),
+                                      dtype_code(out.dtype), out.stride(0), n_seqs, channels, n_states, dt_rank,
+                                      float(out_scale), _stream()), "selective_scan")
+    _launched()
+
+
+def selective_step(u: torch.Tensor, low: torch.Tensor, dt_weight: torch.Tensor, dt_bias: torch.Tensor,
+                   a_log2: torch.Tensor, d: torch.Tensor, z: torch.Tensor, state: torch.Tensor, state_offset: int,
+                   cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor, n_states: int,
+                   dt_rank: int, out_scale: float = 1.0) -> None:
+    """``selective_scan`` for steps in which every sequence brings at most one token, with ``raw = low[:, :dt_rank] @
+    dt_weight.T`` (``dt_weight`` [channels, dt_rank] in the activation dtype) folded in."""
+    n, channels = _scan_operands(u, low, dt_bias, a_log2, d, z, state, state_offset, out, n_states, dt_rank)
+    _need(dt_weight, "dt_weight", u.dtype)
+    assert tuple(dt_weight.shape) == (channels, dt_rank)
+    check(library().mx_selective_step(_ptr(u), _ptr(low), low.stride(0), _ptr(dt_weight), _ptr(dt_bias), _ptr(a_log2),
+                                      _ptr(d), _ptr(z), dtype_code(z.dtype), z.stride(0), _ptr(state), state.stride(0),
+                                      int(state_offset), _ptr(cu_q), _ptr(state_slots), _ptr(out), dtype_code(out.dtype),
+                                      out.stride(0), n_seqs, channels, n_states, dt_rank, float(out_scale), _stream()),
+          "selective_step")
+    _launched()
+
+
+def cast_columns(x: torch.Tensor, out: torch.Tensor) -> None:
+    """out (bfloat16, contiguous) = x (a float32 column range of wider rows)."""
+    _need(x, "x", torch.float32, contiguous=False)
+    _need(out, "out", torch.bfloat16)
+    n, width = out.shape
+    assert tuple(x.shape) == (n, width) and x.stride(1) == 1
+    check(library().mx_cast_columns(_ptr(x), x.stride(0), _ptr(out), n, width, _stream()), "cast_columns")
     _launched()

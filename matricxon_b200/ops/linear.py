@@ -26,6 +26,7 @@ from matricxon_b200.ops.kernels import (
     EPILOGUE_F32,
     EPILOGUE_GELU,
     EPILOGUE_NONE,
+    EPILOGUE_RELU2,
     EPILOGUE_RESIDUAL,
 )
 from matricxon_b200.ops.library import KernelLibraryError
@@ -129,7 +130,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, mod
            backend: str = "auto", defer_sum: bool = False) -> "torch.Tensor | PendingSum":
     """x [M, K], weight [N, K] in the compute dtype; bias float32 [N] or None.
 
-    mode EPILOGUE_NONE / EPILOGUE_GELU give the compute dtype; EPILOGUE_RESIDUAL
+    mode EPILOGUE_NONE / EPILOGUE_GELU / EPILOGUE_RELU2 (the square of relu) give the compute dtype; EPILOGUE_RESIDUAL
     (``residual + x @ W.T + bias``) and EPILOGUE_F32 give float32.
 
     ``defer_sum`` (EPILOGUE_RESIDUAL into the residual itself): where the product is the library's, the
@@ -228,4 +229,4 @@ def _bmm(a: torch.Tensor, b: torch.Tensor, out_dtype: torch.dtype) -> torch.Tens
 
 
 __all__ = ["linear", "batched_linear", "chosen_backend", "PendingSum", "resolve_backend", "EPILOGUE_NONE", "EPILOGUE_GELU", "EPILOGUE_RESIDUAL",
-           "EPILOGUE_F32"]
+           "EPILOGUE_F32", "EPILOGUE_RELU2"]

@@ -1,9 +1,11 @@
 """Parts a model is assembled from. Importing this package registers the built-in kinds."""
 
 from matricxon_b200.parts import (  # noqa: F401  (registration)
-    attention, block, latent_attention, linear_attention, mlp, norm, pass_input, recurrent, rotary, routed, side_input)
+    attention, block, latent_attention, linear_attention, mlp, norm, parallel, pass_input, recurrent, rotary, routed,
+    selective, side_input)
 from matricxon_b200.parts.base import (
     Block,
+    BranchMixer,
     CacheBinding,
     FeedForward,
     KVCacheRequest,
@@ -18,6 +20,6 @@ from matricxon_b200.parts.base import (
     register_part,
 )
 
-__all__ = ["Block", "CacheBinding", "FeedForward", "KVCacheRequest", "Mixer", "Norm", "Part",
+__all__ = ["Block", "BranchMixer", "CacheBinding", "FeedForward", "KVCacheRequest", "Mixer", "Norm", "Part",
            "PositionEncoding", "Runtime", "StateRequest", "build_part", "part_class",
            "register_part"]

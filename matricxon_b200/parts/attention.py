@@ -24,7 +24,7 @@ import torch
 
 from matricxon_b200.ops import kernels
 from matricxon_b200.ops.linear import EPILOGUE_F32, EPILOGUE_NONE, EPILOGUE_RESIDUAL, chosen_backend, linear
-from matricxon_b200.parts.base import KVCacheRequest, Mixer, build_part, register_part
+from matricxon_b200.parts.base import BranchMixer, KVCacheRequest, Mixer, StateRequest, build_part, register_part
 from matricxon_b200.parts.rotary import store_without_rotation
 from matricxon_b200.weights.loader import WeightSpec
 
@@ -115,7 +115,7 @@ def simt_splits(ctx, n_heads: int, n_kv_heads: int, head_dim: int, window: int |
 
 
 def paged_attend(q, q_stride, ctx, binding, rt, n_heads, n_kv_heads, head_dim, window, scale, softcap=None,
-                 sink=None, keep_first=0, chunk=None):
+                 sink=None, keep_first=0, chunk=None, distance=None, out=None):
     """Attention of the step's query rows (``q``: query head h of a row at column ``h * head_dim``, rows
     ``q_stride`` apart) over the keys and values already stored in ``binding.kv``: picks the kernel, the
     tiles and the key splits for this step. Returns [tokens, heads * head_dim] in the runtime dtype.
@@ -123,8 +123,9 @@ def paged_attend(q, q_stride, ctx, binding, rt, n_heads, n_kv_heads, head_dim, w
     head) joins the softmax's denominator without a value. ``keep_first``: under a window, the keys of the
     sequence's first ``keep_first`` positions stay visible at any distance. ``chunk`` (instead of a window): the
     sequence is cut into blocks of ``chunk`` positions counted from its start and a query sees the keys of its own
-    block only; the kernels take this rule as a negative ``window``. Every kernel takes cap, sink, kept tokens and
-    blocks."""
+    block only; the kernels take this rule as a negative ``window``. ``distance`` (float32 [2, heads]): the score of
+    the query at p and the key at j loses ``r1_h ln(1 + r2_h (p - j))``. Every kernel takes cap, sink, kept tokens, blocks
+    and distance. ``out``: where the result goes (rows may be strided)."""
     if chunk is not None:
         if window is not None:
             raise ValueError("attention is masked by a window or by blocks, not both")
@@ -132,16 +133,18 @@ def paged_attend(q, q_stride, ctx, binding, rt, n_heads, n_kv_heads, head_dim, w
             raise ValueError(f"blocks hold at least one position, got {chunk}")
         # a query walks at most the keys of one block
         attn = paged_attend(q, q_stride, _SpanLimited(ctx, int(chunk)), binding, rt, n_heads, n_kv_heads, head_dim,
-                            -int(chunk), scale, softcap=softcap, sink=sink)
+                            -int(chunk), scale, softcap=softcap, sink=sink, distance=distance, out=out)
         return attn
     keep_first = int(keep_first) if window is not None and window > 0 else 0
-    extras = {"softcap": softcap, "sink": sink}
+    extras = {"softcap": softcap, "sink": sink, "distance": distance}
     kept = {"keep_first": keep_first}
     # the kept keys are walked beside the window's: the span that sizes the key splits grows by them
     span = None if window is None or window < 0 else window + keep_first
     group = ctx.groups[binding.group]
-    attn = torch.empty((ctx.n_tokens, n_heads * head_dim), dtype=rt.dtype, device=q.device)
-    if kernels.mma_attention_supported(rt.dtype, head_dim, rt.page_size, q_stride):
+    attn = out if out is not None else torch.empty((ctx.n_tokens, n_heads * head_dim), dtype=rt.dtype, device=q.device)
+    # 16-byte stores of the results want aligned rows
+    aligned = attn.stride(0) % 8 == 0 and attn.data_ptr() % 16 == 0
+    if aligned and kernels.mma_attention_supported(rt.dtype, head_dim, rt.page_size, q_stride):
         group_size = n_heads // n_kv_heads
         # prompt portions on tcgen05 when the kernel takes the geometry, else on mma.sync
         on_tc = _TC_ATTENTION and kernels.tc_attention_supported(rt.dtype, head_dim, rt.page_size, q_stride, group_size)
@@ -518,17 +521,18 @@ class UnitNormAttention(Mixer):
 
 
 @register_part("mixer", "normed_rotary_attention")
-class NormedRotaryAttention(Mixer):
+class NormedRotaryAttention(BranchMixer):
     """Grouped-query attention without biases whose queries and keys are RMS-normalised head by head with a learned
     weight and then rotated over their first entries; causal, windowed or cut into blocks; with an ordinary softmax,
     one added to its denominator, or a learned sink; optionally capped scores; a sigmoid gate per head or per entry
     that reads the mixer's input (``NormedRotaryAttentionSpec``).
 
-    One fused product gives float rows ``[q | k | v | gate]``; one kernel normalises and rotates q and k in float and
-    stores k and v in the paged cache in the layout the stock attention kernels read (``paged_attend``, which knows
-    every mask, the cap and the sink), every head padded with zeros to a common size of a multiple of 16 when the key
-    and value widths differ or are no such multiple; one kernel applies the gate and drops the padding.
-    ``forward(h, None, ...)`` returns the mixer's float output without a residual."""
+    One fused product gives float rows ``[q | k | v | gate]`` (``[q | k | gate]`` where the values are the keys as
+    projected); one kernel normalises and rotates q and k in float and stores k and v in the paged cache in the layout
+    the stock attention kernels read (``paged_attend``, which knows every mask, the cap and the sink), every head padded
+    with zeros to a common size of a multiple of 16 when the key and value widths differ or are no such multiple; one
+    kernel applies the gate and drops the padding. A scale that the mixer around it asks for goes on the stored values
+    (attention is linear in them). ``forward(h, None, ...)`` returns the mixer's float output without a residual."""
 
     capturable = True
 
@@ -548,8 +552,9 @@ class NormedRotaryAttention(Mixer):
     @classmethod
     def _matrices(cls, spec):
         shapes = [(spec.query_name, (spec.num_heads * spec.head_dim, spec.hidden_size)),
-                  (spec.key_name, (spec.num_kv_heads * spec.head_dim, spec.hidden_size)),
-                  (spec.value_name, (spec.num_kv_heads * spec.value_dim, spec.hidden_size))]
+                  (spec.key_name, (spec.num_kv_heads * spec.head_dim, spec.hidden_size))]
+        if spec.value_name is not None:
+            shapes.append((spec.value_name, (spec.num_kv_heads * spec.value_dim, spec.hidden_size)))
         if spec.gate == "head":
             shapes.append((spec.gate_name, (spec.num_heads, spec.hidden_size)))
         elif spec.gate == "entry":
@@ -577,8 +582,8 @@ class NormedRotaryAttention(Mixer):
 
     def load(self, fetch):
         p, s = self.prefix, self.spec
-        self.proj_weight = torch.cat([fetch(p + name) for name, _ in self._matrices(s)])
-        self.o_weight = fetch(p + s.output_name)
+        self.input_weight = torch.cat([fetch(p + name) for name, _ in self._matrices(s)])
+        self.output_weight = fetch(p + s.output_name)
         self.q_norm = fetch(p + s.query_norm_name) if s.query_norm_name is not None else None
         self.k_norm = fetch(p + s.key_norm_name) if s.key_norm_name is not None else None
         if s.sink == "learned":
@@ -588,38 +593,161 @@ class NormedRotaryAttention(Mixer):
         else:
             self.sink = None
 
+    def mix(self, proj, ctx, binding, out, scale=1.0):
+        s, rt, hd = self.spec, self.runtime, self.padded_dim
+        if binding.kv is None:
+            raise RuntimeError("attention needs cache pages bound to it")
+        n = proj.shape[0]
+        q = torch.empty((n, s.num_heads * hd), dtype=rt.dtype, device=proj.device)
+        writes = binding.writes
+        if scale != 1.0 and not writes:
+            raise RuntimeError("a scaled branch stores its values itself")
+        if self.position is not None:
+            freq, rot = self.position.frequencies, s.position.rotary_dim
+            interleaved = bool(getattr(self.position, "interleaved", False))
+            amplitude = float(getattr(self.position, "amplitude", 1.0))
+        else:
+            freq, rot, interleaved, amplitude = torch.empty(0, dtype=torch.float32, device=proj.device), 0, False, 1.0
+        kernels.norm_rotate_kv_write(proj, ctx.positions, freq, rot, interleaved, self.q_norm, self.k_norm, s.eps,
+                                     ctx.groups[binding.group].slots if writes else None,
+                                     binding.kv if writes else None, q, s.num_heads, s.num_kv_heads, s.head_dim,
+                                     s.value_dim, ctx.status, amplitude=amplitude, values_are_keys=s.value_name is None,
+                                     value_scale=scale)
+        direct = s.gate is None and hd == s.value_dim          # nothing stands between the kernel and the output product
+        attn = paged_attend(q, q.stride(0), ctx, binding, rt, s.num_heads, s.num_kv_heads, hd,
+                            s.mask_size if s.mask == "window" else None, s.scale, softcap=s.softcap, sink=self.sink,
+                            chunk=s.mask_size if s.mask == "chunk" else None, out=out if direct else None)
+        if direct:
+            return
+        if s.gate is None:
+            out.view(n, s.num_heads, s.value_dim).copy_(attn.view(n, s.num_heads, hd)[:, :, :s.value_dim])
+            return
+        gate_col = (s.num_heads + s.num_kv_heads) * s.head_dim
+        if s.value_name is not None:
+            gate_col += s.num_kv_heads * s.value_dim
+        gate = proj[:, gate_col:gate_col + self.gate_rows]
+        gated = out if out.is_contiguous() else torch.empty(tuple(out.shape), dtype=rt.dtype, device=out.device)
+        if s.gate == "head":
+            kernels.head_gate(attn, gate, gated, s.num_heads, s.value_dim)
+        else:
+            kernels.sigmoid_gate(attn, gate, gated, s.num_heads, s.value_dim)
+        if gated is not out:
+            out.copy_(gated)
+
+
+@register_part("mixer", "conv_attention")
+class ConvAttention(Mixer):
+    """Causal grouped-query attention behind short convolutions, with queries and keys normalised over the whole
+    projection, a query temperature that grows with the position and a bias on the scores that grows with the logarithm
+    of the distance; it may attend over an earlier layer's keys and values (``ConvAttentionSpec``).
+
+    One fused product gives float rows ``[q | k | v]`` (``[q]`` where the cache is another layer's); one kernel adds the
+    biases, convolves, normalises, puts the temperature on q and stores k and v in the paged cache in the layout the
+    stock attention kernels read (``paged_attend``, which knows the distance bias), every head padded with zeros to a
+    common size of a multiple of 16 when the key and value widths differ or are no such multiple. Per request the state
+    slot holds the latest ``taps - 1`` rows ``[q | k | v]`` with their biases, float32. The keys that a sharing layer
+    reads are those of its source's cache: convolved and normalised; the values convolved only."""
+
+    capturable = True
+
+    def __init__(self, spec, runtime, prefix):
+        super().__init__(spec, runtime, prefix)
+        self.padded_dim = self.cache_head_dim(spec)
+        self.temperature = spec.temperature if spec.temperature is not None else (0.0, 1.0)
+
+    @staticmethod
+    def cache_head_dim(spec) -> int:
+        return -(-max(spec.head_dim, spec.value_dim) // 16) * 16
+
+    @classmethod
+    def _projections(cls, spec):
+        """(name, rows) of the projections, in the order of the fused product's rows."""
+        rows = [(spec.query_name, spec.num_heads * spec.head_dim)]
+        if not spec.shares_kv:
+            rows += [(spec.key_name, spec.num_kv_heads * spec.head_dim),
+                     (spec.value_name, spec.num_kv_heads * spec.value_dim)]
+        return rows
+
+    @classmethod
+    def weight_specs(cls, spec, prefix):
+        specs = []
+        for name, rows in cls._projections(spec):
+            specs.append(WeightSpec(prefix + name, (rows, spec.hidden_size), role="matrix", init="weight"))
+            if spec.bias:
+                specs.append(WeightSpec(prefix + name + spec.bias_suffix, (rows,), role="vector", init="bias"))
+            if spec.taps is not None:
+                specs.append(WeightSpec(prefix + name + spec.conv_suffix, (rows, spec.taps), role="vector", init="weight"))
+        specs.append(WeightSpec(prefix + spec.query_norm_name, (spec.num_heads * spec.head_dim,), role="vector",
+                                init="norm_weight"))
+        if not spec.shares_kv:
+            specs.append(WeightSpec(prefix + spec.key_norm_name, (spec.num_kv_heads * spec.head_dim,), role="vector",
+                                    init="norm_weight"))
+        for name in spec.distance_names or ():
+            specs.append(WeightSpec(prefix + name, (spec.num_heads,), role="vector", init="norm_weight"))
+        specs.append(WeightSpec(prefix + spec.output_name, (spec.hidden_size, spec.num_heads * spec.value_dim),
+                                role="matrix", init="weight"))
+        if spec.bias:
+            specs.append(WeightSpec(prefix + spec.output_name + spec.bias_suffix, (spec.hidden_size,), role="vector",
+                                    init="bias"))
+        return specs
+
+    @classmethod
+    def cache_request(cls, spec):
+        return KVCacheRequest(num_kv_heads=spec.num_kv_heads, head_dim=cls.cache_head_dim(spec), window=None)
+
+    @classmethod
+    def state_request(cls, spec):
+        if spec.taps is None or spec.taps == 1:
+            return None
+        return StateRequest(shape=(spec.taps - 1, sum(rows for _, rows in cls._projections(spec))), dtype=torch.float32)
+
+    def load(self, fetch):
+        p, s = self.prefix, self.spec
+        projections = self._projections(s)
+        self.proj_weight = torch.cat([fetch(p + name) for name, _ in projections])
+        self.proj_bias = torch.cat([fetch(p + name + s.bias_suffix) for name, _ in projections]) if s.bias else None
+        if s.taps is not None:
+            # [taps][channels]: a tap's weights of neighbouring channels lie side by side
+            self.conv = torch.cat([fetch(p + name + s.conv_suffix) for name, _ in projections]).t().contiguous()
+        else:
+            self.conv = torch.ones((1, self.proj_weight.shape[0]), dtype=torch.float32, device=self.runtime.device)
+        self.q_norm = fetch(p + s.query_norm_name)
+        self.k_norm = fetch(p + s.key_norm_name) if not s.shares_kv else None
+        self.distance = (torch.stack([fetch(p + name) for name in s.distance_names]).contiguous()
+                         if s.distance_names is not None else None)
+        self.o_weight = fetch(p + s.output_name)
+        self.o_bias = fetch(p + s.output_name + s.bias_suffix) if s.bias else None
+
     def forward(self, h, residual, ctx, binding):
         s, rt, hd = self.spec, self.runtime, self.padded_dim
         if binding.kv is None:
             raise RuntimeError("attention needs cache pages bound to it")
-        n = h.shape[0]
+        if s.shares_kv == binding.writes:
+            raise RuntimeError("a layer owns its cache exactly if it has key and value projections")
+        taps = self.conv.shape[0]
+        if taps > 1 and binding.state is None:
+            raise RuntimeError("the convolutions need a state tensor bound to them")
+        n, channels = h.shape[0], self.proj_weight.shape[0]
         proj = linear(h, self.proj_weight, None, EPILOGUE_F32, backend=rt.gemm_backend)
         q = torch.empty((n, s.num_heads * hd), dtype=rt.dtype, device=h.device)
-        writes = binding.writes
-        if self.position is not None:
-            freq, rot = self.position.frequencies, s.position.rotary_dim
-            interleaved = bool(getattr(self.position, "interleaved", False))
-        else:
-            freq, rot, interleaved = torch.empty(0, dtype=torch.float32, device=h.device), 0, False
-        kernels.norm_rotate_kv_write(proj, ctx.positions, freq, rot, interleaved, self.q_norm, self.k_norm, s.eps,
-                                     ctx.groups[binding.group].slots if writes else None,
-                                     binding.kv if writes else None, q, s.num_heads, s.num_kv_heads, s.head_dim,
-                                     s.value_dim, ctx.status)
-        attn = paged_attend(q, q.stride(0), ctx, binding, rt, s.num_heads, s.num_kv_heads, hd,
-                            s.mask_size if s.mask == "window" else None, s.scale, softcap=s.softcap, sink=self.sink,
-                            chunk=s.mask_size if s.mask == "chunk" else None)
-        if s.gate is not None:
-            gate_col = (s.num_heads + s.num_kv_heads) * s.head_dim + s.num_kv_heads * s.value_dim
-            gated = torch.empty((n, s.num_heads * s.value_dim), dtype=rt.dtype, device=h.device)
-            gate = proj[:, gate_col:gate_col + self.gate_rows]
-            if s.gate == "head":
-                kernels.head_gate(attn, gate, gated, s.num_heads, s.value_dim)
-            else:
-                kernels.sigmoid_gate(attn, gate, gated, s.num_heads, s.value_dim)
-            attn = gated
-        elif hd != s.value_dim:
+        kernels.conv_norm_kv_write(proj, self.proj_bias, self.conv, self.q_norm, self.k_norm, s.eps, self.temperature,
+                                   binding.state, ctx.positions, ctx.tok_seq, ctx.cu_q, ctx.state_slots,
+                                   ctx.groups[binding.group].slots if binding.writes else None,
+                                   binding.kv if binding.writes else None, q, s.num_heads, s.num_kv_heads, s.head_dim,
+                                   s.value_dim, ctx.status)
+        if taps > 1 and not one_token_each(ctx):
+            kernels.conv_state_update(proj, self.proj_bias, binding.state.flatten(1), ctx.cu_q, ctx.state_slots, ctx.n_seqs,
+                                      channels, taps)
+        attn = paged_attend(q, q.stride(0), ctx, binding, rt, s.num_heads, s.num_kv_heads, hd, None, s.scale,
+                            distance=self.distance)
+        if hd != s.value_dim:
             attn = attn.view(n, s.num_heads, hd)[:, :, :s.value_dim].reshape(n, -1)
         if residual is None:
-            return linear(attn, self.o_weight, None, EPILOGUE_F32, backend=rt.gemm_backend)
-        return linear(attn, self.o_weight, None, EPILOGUE_RESIDUAL, residual=residual, out=residual,
+            return linear(attn, self.o_weight, self.o_bias, EPILOGUE_F32, backend=rt.gemm_backend)
+        return linear(attn, self.o_weight, self.o_bias, EPILOGUE_RESIDUAL, residual=residual, out=residual,
                       backend=rt.gemm_backend, defer_sum=getattr(ctx, "sums_may_pend", False))
+
+
+def one_token_each(ctx) -> bool:
+    """Whether no sequence of the step brings more than one token (known on the host, whatever the step replays)."""
+    return ctx.padded or max(ctx.host.q_lens) <= 1

@@ -15,6 +15,7 @@ Interfaces (duck-typed; these base classes state them):
       encodes q (and k) inside ``qkv`` in place and stores k, v into the bound cache pages.
   Mixer.forward(h, residual, ctx, binding) -> residual + mix(h)      (float32)
   Mixer.cache_request(spec) / Mixer.state_request(spec): what the cache manager must hold.
+  BranchMixer.input_weight, .mix(proj, ctx, binding, out, scale), .output_weight: a mixer that can stand beside others
   FeedForward.forward(h, residual, ctx) -> residual + ffn(h)          (float32)
   SideInput.forward(x, h, ctx) -> (x, activations)                     (x updated in place; h = x in the runtime dtype)
   PassInput.begin(x0, ctx); PassInput.forward(x, pass_index, ctx) -> x  (before the entry that opens a pass)
@@ -176,6 +177,36 @@ class Mixer(Part):
 
     def forward(self, h, residual, ctx, binding):
         raise NotImplementedError
+
+
+class BranchMixer(Mixer):
+    """A mixer that can stand beside others on the same input (``ParallelMixerSpec``). It is cut where its two large
+    products are: ``input_weight`` ([rows, hidden], one product of the input), then ``mix``, then ``output_weight``
+    ([hidden, columns]). Alone it runs all three (``forward``); side by side, the mixer around it makes one input and
+    one output product for all branches and calls ``mix`` in between.
+
+    ``mix(proj, ctx, binding, out, scale)`` fills ``out`` [tokens, output columns] (runtime dtype, rows may be strided)
+    with ``scale`` times what the output product reads, from the float rows ``proj`` of the input product."""
+
+    input_weight = None
+    output_weight = None
+
+    def mix(self, proj, ctx, binding, out, scale=1.0):
+        raise NotImplementedError
+
+    def forward(self, h, residual, ctx, binding):
+        import torch
+
+        from matricxon_b200.ops.linear import EPILOGUE_F32, EPILOGUE_RESIDUAL, linear
+
+        rt = self.runtime
+        proj = linear(h, self.input_weight, None, EPILOGUE_F32, backend=rt.gemm_backend)
+        mixed = torch.empty((h.shape[0], self.output_weight.shape[1]), dtype=rt.dtype, device=h.device)
+        self.mix(proj, ctx, binding, mixed)
+        if residual is None:
+            return linear(mixed, self.output_weight, None, EPILOGUE_F32, backend=rt.gemm_backend)
+        return linear(mixed, self.output_weight, None, EPILOGUE_RESIDUAL, residual=residual, out=residual,
+                      backend=rt.gemm_backend, defer_sum=getattr(ctx, "sums_may_pend", False))
 
 
 class FeedForward(Part):

@@ -1,5 +1,6 @@
-"""Gated linear attention: a matrix state per head that decays per key channel.
+"""Linear attention: a matrix state per head that decays.
 
+Gated linear attention decays per key channel, by the token.
 Per token t and head (``GlaSpec``): ``q = Wq h * query_scale``, ``k = Wk h``, ``v = Wv h``, a decay per key channel
 ``a = sigmoid(A2 (A1 h) + b)^(1/tau)``; ``S_t = diag(a_t) S_(t-1) + k_t v_t^T`` from S = 0 and ``o_t = S_t^T q_t``.
 Every head's o is RMS-normalised over its value width with one plain weight, multiplied by ``silu(Wg h)`` and
@@ -9,6 +10,11 @@ it for the next one, so a sequence may be cut anywhere.
 One fused product gives float rows ``[q | k | v | gate | A1 h]``; the second decay product (rank x channels, tiny)
 stays on the FP32 cores with float weights, so the decays, their logarithms and exponentials, the state, the norm
 and the gate are float in both dtypes; only the large projections run in the runtime dtype.
+
+Retention (``RetentionSpec``) decays by one constant per head: ``S_t = decay_h S_(t-1) + k_t v_t^T``, ``o_t = S_t^T q_t`` with
+q and k rotated over their first entries. It shares the recurrence's kernel (which takes no decay operand then), the
+state's layout and the kernel behind it (no weight in its norm). Long portions are rotated by a pass of their own, steps
+of one token a sequence on the operands' way into the recurrence.
 """
 
 from __future__ import annotations
@@ -17,7 +23,8 @@ import torch
 
 from matricxon_b200.ops import kernels
 from matricxon_b200.ops.linear import EPILOGUE_F32, EPILOGUE_RESIDUAL, linear
-from matricxon_b200.parts.base import Mixer, StateRequest, register_part
+from matricxon_b200.parts.attention import one_token_each
+from matricxon_b200.parts.base import BranchMixer, Mixer, StateRequest, build_part, register_part
 from matricxon_b200.weights.loader import WeightSpec
 
 
@@ -76,3 +83,64 @@ class GatedLinearAttention(Mixer):
             return linear(out, self.o_weight, None, EPILOGUE_F32, backend=rt.gemm_backend)
         return linear(out, self.o_weight, None, EPILOGUE_RESIDUAL, residual=residual, out=residual,
                       backend=rt.gemm_backend, defer_sum=getattr(ctx, "sums_may_pend", False))
+
+
+@register_part("mixer", "retention")
+class Retention(BranchMixer):
+    capturable = True
+
+    def __init__(self, spec, runtime, prefix):
+        super().__init__(spec, runtime, prefix)
+        self.position = (build_part("position", spec.position, runtime, prefix)
+                         if spec.position is not None and spec.position.rotary_dim > 0 else None)
+        if self.position is not None and (not hasattr(self.position, "frequencies")
+                                          or getattr(self.position, "interleaved", False)
+                                          or getattr(self.position, "amplitude", 1.0) != 1.0):
+            raise ValueError(f"retention rotates by a plain table with halves paired, not by {spec.position!r}")
+
+    @classmethod
+    def _matrices(cls, spec):
+        keys, values = spec.num_heads * spec.head_dim, spec.num_heads * spec.value_dim
+        return [(spec.query_name, keys), (spec.key_name, keys), (spec.value_name, values), (spec.gate_name, values)]
+
+    @classmethod
+    def weight_specs(cls, spec, prefix):
+        specs = [WeightSpec(prefix + name, (rows, spec.hidden_size), role="matrix", init="weight")
+                 for name, rows in cls._matrices(spec)]
+        specs.append(WeightSpec(prefix + spec.output_name, (spec.hidden_size, spec.num_heads * spec.value_dim),
+                                role="matrix", init="weight"))
+        return specs
+
+    @classmethod
+    def state_request(cls, spec):
+        return StateRequest(shape=(spec.num_heads, spec.head_dim, spec.value_dim), dtype=torch.float32)
+
+    def load(self, fetch):
+        p, s = self.prefix, self.spec
+        self.input_weight = torch.cat([fetch(p + name) for name, _ in self._matrices(s)])
+        self.output_weight = fetch(p + s.output_name)
+        self.decay = torch.tensor(s.decay, dtype=torch.float32, device=self.runtime.device)
+
+    def mix(self, proj, ctx, binding, out, scale=1.0):
+        s = self.spec
+        if binding.state is None:
+            raise RuntimeError("retention needs a state tensor bound to it")
+        if scale != 1.0:
+            raise RuntimeError("retention's output is normalised per head: it takes no scale")
+        n, keys, values = proj.shape[0], s.num_heads * s.head_dim, s.num_heads * s.value_dim
+        rotation = {}
+        if self.position is not None:
+            freq, rot = self.position.frequencies, s.position.rotary_dim
+            if one_token_each(ctx):
+                rotation = {"positions": ctx.positions, "freq": freq, "rot": rot}
+            else:                                                     # q and k heads lie side by side
+                kernels.rotate_heads(proj, 0, 2 * s.num_heads, s.head_dim, rot, ctx.positions, freq)
+        o = torch.empty((n, values), dtype=torch.float32, device=proj.device)
+        # the scale of k goes on q: the output is linear in both, and the state then holds the plain k v^T
+        kernels.retention_scan(proj, 0, keys, 2 * keys, self.decay, s.key_scale, binding.state, ctx.cu_q, ctx.state_slots,
+                               ctx.n_seqs, o, s.num_heads, s.head_dim, s.value_dim, **rotation)
+        gate = proj[:, 2 * keys + values:2 * keys + 2 * values]
+        rows = out if out.is_contiguous() else torch.empty(tuple(out.shape), dtype=out.dtype, device=out.device)
+        kernels.gla_norm_gate(o, gate, None, s.eps, rows, s.num_heads, s.value_dim)
+        if rows is not out:
+            out.copy_(rows)

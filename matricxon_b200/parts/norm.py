@@ -64,18 +64,22 @@ class RmsNorm(Norm):
     """``x / sqrt(mean(x^2) + eps) * scale`` with float statistics; the stored weight is the scale or,
     with ``unit_offset``, the scale minus one. Beside the plain form it ends a post-norm sublayer in one
     kernel: ``forward_scaled_sum`` forms ``skip_scale * x + sublayer``, normalises it into the residual
-    stream and hands the next sublayer its input in the runtime dtype."""
+    stream and hands the next sublayer its input in the runtime dtype. Like LayerNorm it can form a residual sum that a
+    library product left unadded on its way through the rows. A scale of one number (``scalar``) is held as a vector."""
 
     capturable = True
+    adds_pending_sum = True
 
     @classmethod
     def weight_specs(cls, spec, prefix):
         # a weight stored around zero is drawn like a norm's shift when random weights are asked for
         init = "norm_bias" if spec.unit_offset else "norm_weight"
-        return [WeightSpec(prefix + spec.weight_name, (spec.size,), role="vector", init=init)]
+        return [WeightSpec(prefix + spec.weight_name, () if spec.scalar else (spec.size,), role="vector", init=init)]
 
     def load(self, fetch):
         self.weight = fetch(self.prefix + self.spec.weight_name)
+        if self.spec.scalar:
+            self.weight = self.weight.reshape(1).expand(self.spec.size).contiguous()
         self.offset = 1.0 if self.spec.unit_offset else 0.0
         self.scale = self.weight + 1.0 if self.spec.unit_offset else self.weight      # what a row is multiplied with
 
@@ -85,6 +89,14 @@ class RmsNorm(Norm):
             out = torch.empty((n_rows, self.spec.size), dtype=self.runtime.dtype, device=x.device)
         kernels.rmsnorm(x, self.weight, self.offset, self.spec.eps, out, rows)
         return out
+
+    def forward_sum(self, pending):
+        """The norm of a residual sum that has not been added up yet (``ops.linear.PendingSum``), formed by the same
+        kernel. Returns (x, norm(x))."""
+        x = pending.added_by_kernel()
+        out = torch.empty(tuple(x.shape), dtype=self.runtime.dtype, device=x.device)
+        kernels.rmsnorm_pending(x, pending.acc, pending.bias, self.weight, self.offset, self.spec.eps, out)
+        return x, out
 
     def forward_scaled_sum(self, x, sublayer, skip_scale):
         """``x <- norm(skip_scale * x + sublayer)`` in place (both float32). Returns (x, activations): the

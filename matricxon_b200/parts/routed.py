@@ -17,7 +17,8 @@ second weighs every pair's row). The experts' matrices are stacked at load: ``[e
 the weights; optionally a bias on the logits themselves, which makes the rule "the largest logits, weighted by the
 softmax over the chosen ones") and may name experts without matrices that return their input: such a pair takes no row of the grouped
 products, and the combining kernel adds ``weight * h`` for it. An expert may be a ``GatedMlpSpec`` or a
-``ClampedGluSpec`` (the activation differs). A ``shared`` feed-forward runs for every token; the routed sum is added
+``ClampedGluSpec`` (the activation differs). ``weight_on="input"`` puts a pair's weight on the expert's input instead of
+its output, ``normalize=False`` leaves the sigmoid scores as the weights. A ``shared`` feed-forward runs for every token; the routed sum is added
 onto its output.
 """
 
@@ -104,7 +105,7 @@ class RoutedExperts(FeedForward):
                                       bias=self.bias)
         else:
             kernels.moe_route(h, self.router, s.top, s.num_groups, s.groups_kept, s.route_scale, ids, weights, counts,
-                              place)
+                              place, normalize=s.normalize)
         choices = ctx.memo.get("expert_choices") if hasattr(ctx, "memo") else None
         if choices is not None:            # a caller listens (``StepRunner.taps``)
             choices.append(ids.view(n, s.top).clone())
@@ -117,6 +118,9 @@ class RoutedExperts(FeedForward):
         elif residual is None:
             residual = torch.zeros((n, s.hidden_size), dtype=torch.float32, device=device)
         identity = (h, s.num_experts) if s.num_identity else None
+        # a weighted input: both first products are linear, so the weight goes on their results, ahead of the activation
+        before = weights if s.weight_on == "input" else None
+        after = weights if before is None else None
         if on_tc:
             status = getattr(ctx, "status", None)
             rows = torch.empty((n_pairs, s.hidden_size), dtype=h.dtype, device=device)
@@ -127,16 +131,17 @@ class RoutedExperts(FeedForward):
             if self.clamped is not None:
                 kernels.clamped_glu(gate_up, mid, *self.clamped)
             else:
-                kernels.glu(gate_up, mid, e.activation)
+                kernels.glu(gate_up, mid, e.activation, pair_weight=before, order=order if before is not None else None)
             down = torch.empty((n_pairs, s.hidden_size), dtype=torch.float32, device=device)
             kernels.gemm_tcgen05_grouped(mid, self.down, tile_map, n_tiles, max_tiles, down, status)
-            kernels.moe_combine_sorted(down, ids, place, first, weights, residual, s.top, identity=identity)
+            kernels.moe_combine_sorted(down, ids, place, first, after, residual, s.top, identity=identity)
             return residual
         mid = torch.empty((n_pairs, e.intermediate_size), dtype=h.dtype, device=device)
         activation = ("clamped", *self.clamped) if self.clamped is not None else e.activation
-        kernels.moe_gemm(h, order, s.top, self.gate_up, tile_map, n_tiles, max_tiles, mid, None, activation)
+        kernels.moe_gemm(h, order, s.top, self.gate_up, tile_map, n_tiles, max_tiles, mid, None, activation,
+                         input_weight=before)
         pairs = torch.empty((n_pairs, s.hidden_size), dtype=torch.float32, device=device)
-        kernels.moe_gemm(mid, order, 1, self.down, tile_map, n_tiles, max_tiles, pairs, weights, None)
+        kernels.moe_gemm(mid, order, 1, self.down, tile_map, n_tiles, max_tiles, pairs, after, None)
         kernels.moe_combine(pairs, residual, s.top,
                             identity=(ids, weights, h, s.num_experts) if s.num_identity else None)
         return residual

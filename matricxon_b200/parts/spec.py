@@ -81,7 +81,7 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class MlpSpec:
-    """``down(act(up(x)))`` without a gate."""
+    """``down(act(up(x)))`` without a gate; ``activation`` is ``gelu_tanh`` or ``relu_squared``."""
 
     hidden_size: int
     intermediate_size: int
@@ -89,6 +89,8 @@ class MlpSpec:
     activation: str
     up_name: str                 # tensor names under the feed-forward's prefix
     down_name: str
+    weight_suffix: str = ".weight"
+    bias_suffix: str = ".bias"
     kind: str = "mlp"
 
 
@@ -96,12 +98,14 @@ class MlpSpec:
 class RmsNormSpec:
     """``x / sqrt(mean(x^2) + eps) * scale`` over the last axis, eps inside the root. ``unit_offset``:
     the checkpoint stores ``scale - 1`` (a weight around zero). The tensor is called
-    ``<prefix><weight_name>``; an empty ``weight_name`` makes the prefix itself the tensor's name."""
+    ``<prefix><weight_name>``; an empty ``weight_name`` makes the prefix itself the tensor's name. ``scalar``: the
+    scale is one number for all entries (a tensor without axes)."""
 
     size: int
     eps: float
     unit_offset: bool = False
     weight_name: str = "weight"
+    scalar: bool = False
     kind: str = "rmsnorm"
 
 
@@ -439,7 +443,10 @@ class NormedRotaryAttentionSpec:
     counted from its start, and a query sees its own block only). ``sink``: ``None`` for the ordinary softmax,
     ``"zero"`` for a denominator with one added (a logit of 0 without a value), ``"learned"`` for a learned logit
     per head (``sink_name``). ``gate``: ``None``, ``"head"`` (head h times ``sigmoid(G h)_h``, G has one row per head)
-    or ``"entry"`` (the concatenated heads times ``sigmoid(G h)`` entry by entry); the gate reads the mixer's input."""
+    or ``"entry"`` (the concatenated heads times ``sigmoid(G h)`` entry by entry); the gate reads the mixer's input.
+
+    ``position`` may also be an ``InterpolatedRotarySpec`` (its amplitude is then put on cos and sin). ``value_name``
+    None: the values are the keys as projected, before norm and rotation (``value_dim`` equals ``head_dim``)."""
 
     hidden_size: int
     num_heads: int
@@ -451,7 +458,7 @@ class NormedRotaryAttentionSpec:
     position: Any | None
     query_name: str
     key_name: str
-    value_name: str
+    value_name: str | None
     output_name: str
     mask: str = "causal"
     mask_size: int = 0
@@ -470,6 +477,8 @@ class NormedRotaryAttentionSpec:
         if self.head_dim <= 0 or self.value_dim <= 0 or max(self.head_dim, self.value_dim) > 256:
             raise ValueError(f"head sizes {self.head_dim} / {self.value_dim} are outside 1..256: "
                              "no attention kernel of this engine takes them")
+        if self.value_name is None and self.value_dim != self.head_dim:
+            raise ValueError(f"values of {self.value_dim} entries cannot be keys of {self.head_dim}")
         if self.mask not in ("causal", "window", "chunk"):
             raise ValueError(f"mask is 'causal', 'window' or 'chunk', not {self.mask!r}")
         if self.mask != "causal" and self.mask_size <= 0:
@@ -482,6 +491,132 @@ class NormedRotaryAttentionSpec:
             raise ValueError(f"{self.position.rotary_dim} rotated entries exceed the head of {self.head_dim}")
         if self.softcap is not None and not self.softcap > 0:
             raise ValueError(f"a score cap must be positive, got {self.softcap}")
+
+
+@dataclass(frozen=True)
+class ConvAttentionSpec:
+    """Causal grouped-query attention whose projections pass a short causal convolution over time and whose queries and
+    keys are RMS-normalised over the whole projection, all heads at once. For each of q, k and v: ``u = W h (+ b)``,
+    ``y_t = sum_j w[:, j] u_(t - taps + 1 + j)`` per channel (zeros before the sequence's start; ``taps`` None: y = u);
+    ``q = n(y_q) * (1 + coef ln(floor((p + 1) / every) + 1))`` at position p (``temperature`` = (coef, every); None:
+    no factor), ``k = n(y_k)``, ``v = y_v`` with n the RMS norm over all of a projection's rows and a plain weight.
+    Positions enter the scores alone: ``q . k * scale - r1_h ln(1 + r2_h (p - j))`` with two learned numbers per query
+    head (``distance_names``; None: no such term), under an ordinary softmax over every j <= p.
+
+    ``shares_kv``: the layer has no key and value projections and attends over an earlier schedule entry's cache
+    (``ScheduleEntry.cache_of``). Per request the convolutions' latest ``taps - 1`` inputs are kept. Names are full tensor
+    names under the mixer's prefix; a projection's bias and convolution are its name with the suffixes."""
+
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    taps: int | None
+    scale: float
+    eps: float
+    temperature: tuple[float, float] | None
+    bias: bool
+    query_name: str
+    key_name: str
+    value_name: str
+    output_name: str
+    query_norm_name: str
+    key_norm_name: str
+    distance_names: tuple[str, str] | None = None
+    shares_kv: bool = False
+    bias_suffix: str = ".b"
+    conv_suffix: str = ".conv"
+    kind: str = "conv_attention"
+
+    def __post_init__(self) -> None:
+        if self.num_kv_heads <= 0 or self.num_heads % self.num_kv_heads != 0:
+            raise ValueError(f"{self.num_heads} attention heads are no multiple of {self.num_kv_heads} kv heads")
+        if self.head_dim <= 0 or self.value_dim <= 0 or max(self.head_dim, self.value_dim) > 256:
+            raise ValueError(f"head sizes {self.head_dim} / {self.value_dim} are outside 1..256: "
+                             "no attention kernel of this engine takes them")
+        if self.taps is not None and self.taps < 1:
+            raise ValueError("the convolution needs at least one tap")
+        if self.temperature is not None and not self.temperature[1] > 0:
+            raise ValueError(f"the query temperature's period must be positive, got {self.temperature[1]}")
+
+
+@dataclass(frozen=True)
+class SelectiveScanSpec:
+    """A selective state-space recurrence (Mamba): ``[x | z] = W_in h``; ``u = silu(conv(x) + b)`` with ``taps`` per
+    channel, the last on the current token; ``[low | B | C] = W_x u`` (``dt_rank`` | ``states`` | ``states``);
+    ``dt = softplus(W_dt low + b_dt)`` per channel; ``A = -exp(A_log)`` [channels, states];
+    ``S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n`` from S = 0, ``y_c = sum_n S[c, n] C_n + D_c u_c``; the output
+    is ``W_o (y * silu(z))``. Biases are the tensor's name with ``bias_suffix``."""
+
+    hidden_size: int
+    channels: int
+    states: int
+    dt_rank: int
+    taps: int
+    input_name: str
+    conv_name: str
+    low_name: str
+    dt_name: str
+    a_log_name: str
+    d_name: str
+    output_name: str
+    bias_suffix: str = ".b"
+    kind: str = "selective_scan"
+
+    def __post_init__(self) -> None:
+        if min(self.channels, self.states, self.dt_rank) <= 0 or self.taps < 1:
+            raise ValueError("a selective recurrence needs positive channel, state and rank counts and at least one tap")
+        if self.states > 128:
+            raise ValueError(f"{self.states} states per channel: the recurrence kernel takes up to 128")
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention with a constant decay per head: q and k (``head_dim`` wide) rotated over their first entries
+    (``position``; None: not), ``k`` times ``key_scale``; ``S <- decay_h S + k_t v_t^T`` from S = 0, ``o_t = S^T q_t``;
+    every head's o is divided by its root mean square over ``value_dim`` (eps inside, no weight), the heads are
+    multiplied by ``silu(W_g h)`` and projected by W_o. No biases."""
+
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    value_dim: int
+    decay: tuple[float, ...]
+    key_scale: float
+    eps: float
+    position: Any | None
+    query_name: str
+    key_name: str
+    value_name: str
+    gate_name: str
+    output_name: str
+    kind: str = "retention"
+
+    def __post_init__(self) -> None:
+        if min(self.num_heads, self.head_dim, self.value_dim) <= 0:
+            raise ValueError("retention needs positive head count and head sizes")
+        if self.head_dim > 256:
+            raise ValueError(f"{self.head_dim} key channels per head: the recurrence kernel takes up to 256")
+        if len(self.decay) != self.num_heads:
+            raise ValueError(f"{len(self.decay)} decays for {self.num_heads} heads")
+        if self.position is not None and self.position.rotary_dim > self.head_dim:
+            raise ValueError(f"{self.position.rotary_dim} rotated entries exceed the head of {self.head_dim}")
+
+
+@dataclass(frozen=True)
+class ParallelMixerSpec:
+    """Mixers side by side on one input: ``sum_i scale_i * branch_i(h)``. ``branches`` holds (spec, scale, the tensor-name
+    fragment under the mixer's prefix) of mixers that offer the branch interface (``parts.base.BranchMixer``); at
+    most one of them owns paged cache and at most one owns state."""
+
+    hidden_size: int
+    branches: tuple[tuple[Any, float, str], ...]
+    kind: str = "parallel"
+
+    def __post_init__(self) -> None:
+        if not self.branches:
+            raise ValueError("a parallel mixer needs at least one branch")
 
 
 @dataclass(frozen=True)
@@ -566,7 +701,10 @@ class RoutedExpertsSpec:
     ``expert`` may be a ``GatedMlpSpec`` or a ``ClampedGluSpec``. ``shared`` (a feed-forward spec, tensors under
     ``<prefix><shared_name>``) runs for every token and is added. With ``bias_name`` the logits are ``R h + b``; the
     softmax rule with such a bias and without a correction is the same as choosing the ``top`` largest logits and
-    weighting them by the softmax over the chosen logits alone."""
+    weighting them by the softmax over the chosen logits alone.
+
+    ``normalize`` False (sigmoid rule): the weights are ``score * route_scale``. ``weight_on="input"``: a chosen expert
+    runs on ``weight * h`` and its output is added as it is (``"output"``: its output is weighted)."""
 
     hidden_size: int
     num_experts: int
@@ -585,11 +723,21 @@ class RoutedExpertsSpec:
     num_identity: int = 0
     shared: Any | None = None
     shared_name: str = "shared."
+    normalize: bool = True
+    weight_on: str = "output"
     kind: str = "routed_experts"
 
     def __post_init__(self) -> None:
         if self.score not in ("sigmoid", "softmax"):
             raise ValueError(f"router scores are 'sigmoid' or 'softmax', not {self.score!r}")
+        if self.weight_on not in ("output", "input"):
+            raise ValueError(f"a weight goes on an expert's 'output' or 'input', not {self.weight_on!r}")
+        if self.weight_on == "input" and self.expert.kind != "gated_mlp":
+            raise ValueError("weighted inputs are built for gated feed-forwards without clamps")
+        if self.weight_on == "input" and self.num_identity:
+            raise ValueError("weighted inputs go with experts that have matrices only")
+        if not self.normalize and self.score != "sigmoid":
+            raise ValueError("weights that are not normalised belong to the sigmoid rule")
         if self.num_identity < 0 or self.num_experts < 0:
             raise ValueError("expert counts cannot be negative")
         if self.score == "sigmoid" and (self.num_identity or self.correction_name is not None
