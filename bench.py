@@ -21,6 +21,8 @@ models (mixed attention and recurrent layers, gated feed-forwards, a float resid
 models (rotated windowed attention, routed experts through the same grouped products, a float residual stream).
 ``--compare kefasun`` does the same for the Kefasun architecture beside Bafusun, the closest of the engine's other
 models (attention in every layer with normalised queries and keys, routed experts, norms on the branches).
+``--compare seredra`` does the same for the Seredra architecture beside Parunex, the closest of the engine's other models
+(attention and recurrent layers in turn, sigmoid-routed experts through the same grouped products).
 """
 
 from __future__ import annotations
@@ -425,6 +427,33 @@ def kefasun_config(size: dict) -> dict:
             "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers}
 
 
+def seredra_config(size: dict) -> dict:
+    """Capped attention beside a selective recurrence (twice the model's width in channels, 16 states each), retention,
+    and attention behind short convolutions in turn, 128-wide heads (over 4 KV heads where they share keys), the second
+    convolved attention on the first one's keys and values; the first layer with a dense ungated feed-forward of the
+    gated one's parameter count, the others with eight gated experts of half the dense width, two per token."""
+    w, h = size["width"], size["width"] // 128
+    dense = {"kind": "dense", "ff": size["ff"] * 3 // 2}
+    routed = {"kind": "moe", "expert": {"ff": size["ff"] // 2}, "router": {"experts": 8, "top": 2}}
+    parallel = {"type": "parallel",
+                "mixer": {"left": {"heads": h, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+                                   "rot": {"base": 1000000.0, "dims": 64,
+                                           "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+                          "left_scale": 1.0, "right": {"inner": 2 * w, "state": 16, "dt_rank": w // 16, "conv": 4},
+                          "right_scale": 1.0}}
+    retention = {"type": "retention",
+                 "mixer": {"heads": h, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 3.0 * i / h) for i in range(h)],
+                           "rot": {"base": 1000000.0, "dims": 128}}}
+    mixer = {"heads": h, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4,
+             "q_temp": {"coef": 0.1, "every": 1024}}
+    attention = {"type": "attention", "mixer": mixer}
+    sharing = {"type": "attention", "mixer": dict(mixer, kv_from=2)}
+    order = [parallel, retention, attention, parallel, retention, sharing, parallel, retention]
+    layers = [dict(layer, mlp=dense if i == 0 else routed) for i, layer in enumerate(order)]
+    return {"architecture": "Seredra", "vocab": COMPARE_VOCAB, "width": w, "embedding": {"scale": 1.0},
+            "norm": {"eps": 1e-5}, "layers": layers}
+
+
 def starcoder2_like(size: dict) -> dict:
     return dict(STARCODER2_3B, num_hidden_layers=COMPARE_LAYERS, hidden_size=size["width"],
                 num_attention_heads=size["width"] // 128, num_key_value_heads=4, head_dim=128,
@@ -522,7 +551,9 @@ def compare_designs(args) -> int:
     clocks.start()
     sizes = [s for s in args.compare_sizes.split(",") if s]
     batches = [int(b) for b in args.compare_batches.split(",")]
-    if args.compare == "kefasun":
+    if args.compare == "seredra":
+        designs = (("seredra", seredra_config), ("parunex", parunex_config))
+    elif args.compare == "kefasun":
         designs = (("kefasun", kefasun_config), ("bafusun", bafusun_config))
     elif args.compare == "bafusun":
         designs = (("bafusun", bafusun_config), ("parunex", parunex_config))
@@ -567,10 +598,10 @@ def main() -> int:
                         help="leave out the 7B and 15B workloads through the scheduler")
     parser.add_argument("--no-graphs", action="store_true",
                         help="launch every kernel of a decode step by itself (for profilers)")
-    parser.add_argument("--compare", choices=["busatar", "parunex", "bafusun", "kefasun"], default=None,
+    parser.add_argument("--compare", choices=["busatar", "parunex", "bafusun", "kefasun", "seredra"], default=None,
                         help="instead of the headline workload: Busatar beside StarCoder2, Parunex beside Busatar, "
-                             "Bafusun beside Parunex, or Kefasun beside Bafusun, at equal layer sizes (prefill and "
-                             "decode throughput at a few sizes)")
+                             "Bafusun beside Parunex, Kefasun beside Bafusun, or Seredra beside Parunex, at equal "
+                             "layer sizes (prefill and decode throughput at a few sizes)")
     parser.add_argument("--compare-only", default=None,
                         help="with --compare: measure only this one of the two designs (for profilers)")
     parser.add_argument("--compare-sizes", default="w1024,w2048")

@@ -98,25 +98,25 @@ moe_route_kernel(const T* __restrict__ h, int ld, const float* __restrict__ rout
                  int* __restrict__ counts, int* __restrict__ place) {
     extern __shared__ __align__(16) float route_s[];
     float* h_s = route_s;                         // [K]
-    float* score = h_s + K;                       // [experts]
-    float* open = score + n_experts;              // [experts]: the score while the expert may still be chosen, else -1
+    float* logit = h_s + K;                       // [experts]
+    float* open = logit + n_experts;              // [experts]: the logit while the expert may still be chosen, else -inf
     float* worth = open + n_experts;              // [groups]
-    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    router_logits(h + (size_t)t * ld, router, K, n_experts, h_s, score);
-    for (int e = tid; e < n_experts; e += blockDim.x) score[e] = 1.0f / (1.0f + expf(-score[e]));
-    __syncthreads();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    router_logits(h + (size_t)t * ld, router, K, n_experts, h_s, logit);
     if (warp != 0) return;
+    // experts are ranked by their logits: the same order as by sigmoid scores, which run out of digits near one
+    auto score_of = [&](int e) { return 1.0f / (1.0f + expf(-logit[e])); };
     const int per = n_experts / n_groups;
     const bool limited = n_groups > 1 && keep < n_groups;
     for (int g = lane; g < n_groups; g += 32) {
         float a = -1.f, b = -1.f;                 // the two largest of the run (scores are positive)
         for (int e = g * per; e < (g + 1) * per; ++e) {
-            const float s = score[e];
+            const float s = score_of(e);
             if (s > a) { b = a; a = s; } else if (s > b) { b = s; }
         }
         worth[g] = a + (per > 1 ? b : 0.f);
     }
-    for (int e = lane; e < n_experts; e += 32) open[e] = limited ? -1.f : score[e];
+    for (int e = lane; e < n_experts; e += 32) open[e] = limited ? -INFINITY : logit[e];
     __syncwarp();
     if (limited) {
         for (int round = 0; round < keep; ++round) {
@@ -128,21 +128,22 @@ moe_route_kernel(const T* __restrict__ h, int ld, const float* __restrict__ rout
             if (i >= n_groups) i = 0;             // nothing comparable left (scores that are no numbers)
             __syncwarp();
             if (lane == 0) worth[i] = -3.f;
-            for (int e = i * per + lane; e < (i + 1) * per; e += 32) open[e] = score[e];
+            for (int e = i * per + lane; e < (i + 1) * per; e += 32) open[e] = logit[e];
             __syncwarp();
         }
     }
     float total = 0.f, mine = 0.f;
     int my_id = 0;
     for (int slot = 0; slot < top; ++slot) {
-        float v = -2.f;
+        float v = -INFINITY;
         int i = 0x7fffffff;
         for (int e = lane; e < n_experts; e += 32)
             if (open[e] > v) { v = open[e]; i = e; }
         arg_best(v, i);
-        if (i >= n_experts) i = 0;                // nothing comparable left (scores that are no numbers)
+        if (i >= n_experts) i = 0;                // nothing comparable left (logits that are no numbers)
         __syncwarp();
-        if (lane == 0) open[i] = -3.f;
+        v = score_of(i);
+        if (lane == 0) open[i] = -INFINITY;
         __syncwarp();
         total += v;
         if (lane == slot % 32 && slot / 32 == 0) { mine = v; my_id = i; }
