@@ -192,3 +192,12 @@ __device__ __forceinline__ float mode_activation(float v, int mode) {
 __device__ __forceinline__ float mode_activation_fast(float v, int mode) {
     return mode == MX_MODE_GELU ? gelu_tanh_fast(v) : (mode == MX_MODE_RELU2 ? relu_squared(v) : v);
 }
+
+// silu of a value that is rounded to T (or meets operands that were): exact for float, from the hardware's exponential
+// and reciprocal (a few units in the last float place) for bfloat16. The argument stays where the quotient has digits:
+// beyond -80 the result is below any bfloat16 step of what it is added to.
+template <typename T> __device__ __forceinline__ float silu_of(float z);
+template <> __device__ __forceinline__ float silu_of<float>(float z) { return z / (1.f + expf(-z)); }
+template <> __device__ __forceinline__ float silu_of<__nv_bfloat16>(float z) {
+    return __fdividef(z, 1.f + __expf(fminf(-z, 80.f)));
+}

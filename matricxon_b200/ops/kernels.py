@@ -889,14 +889,13 @@ def rglru_scan(xy: torch.Tensor, x_col: int, y_col: int, u: torch.Tensor, gates:
 SCAN_CHUNK = 32     # tokens per chunk of the three-launch recurrence
 
 
-def scan_chunk_lists(q_lens: list[int]) -> tuple[list[int], list[int]]:
-    """For ``rglru_scan_chunked``: (sequence, first token) of every chunk of ``SCAN_CHUNK`` tokens,
-    flattened, sequence by sequence, and the index of each sequence's first chunk (one more entry than
-    sequences)."""
+def scan_chunk_lists(q_lens: list[int], size: int = SCAN_CHUNK) -> tuple[list[int], list[int]]:
+    """For the chunked recurrences: (sequence, first token) of every chunk of ``size`` tokens, flattened, sequence by
+    sequence, and the index of each sequence's first chunk (one more entry than sequences)."""
     chunks: list[int] = []
     first = [0]
     for seq, q_len in enumerate(q_lens):
-        for start in range(0, q_len, SCAN_CHUNK):
+        for start in range(0, q_len, size):
             chunks.extend((seq, start))
         first.append(len(chunks) // 2)
     return chunks, first
@@ -1481,6 +1480,45 @@ def retention_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, head_
     _launched()
 
 
+def retention_chunk_tokens() -> int:
+    return int(library().mx_retention_chunk_tokens())
+
+
+def retention_chunked(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_col: int, head_decay: torch.Tensor,
+                      q_scale: float, eps: float, state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor,
+                      n_seqs: int, chunks: torch.Tensor, seq_chunk0: torch.Tensor, n_chunks: int, out: torch.Tensor,
+                      n_heads: int, dim: int, vdim: int, positions: torch.Tensor | None = None,
+                      freq: torch.Tensor | None = None, rot: int = 0) -> None:
+    """``retention_scan`` and ``gla_norm_gate`` (without a weight) for long portions, in chunks of
+    ``retention_chunk_tokens()`` tokens (``scan_chunk_lists`` on the device) whose products run in parallel on the FP32
+    cores: ``out`` [tokens, heads * vdim] (any activation dtype, rows may be strided) = unit(o) * silu(gate), ``gate`` being
+    the columns from ``g_col`` of the float rows ``proj``. Heads of at most 128 x 128."""
+    for name, tensor in (("proj", proj), ("head_decay", head_decay), ("state", state)):
+        _need(tensor, name, torch.float32, contiguous=name != "proj")
+    for name, tensor in (("chunks", chunks), ("seq_chunk0", seq_chunk0), ("cu_q", cu_q), ("state_slots", state_slots)):
+        _need(tensor, name, torch.int32)
+    _need(out, "out", contiguous=False)
+    n = proj.shape[0]
+    assert tuple(state.shape[1:]) == (n_heads, dim, vdim), state.shape
+    assert proj.stride(1) == 1 and proj.shape[1] >= g_col + n_heads * vdim and head_decay.numel() == n_heads
+    assert tuple(out.shape) == (n, n_heads * vdim) and out.stride(1) == 1
+    assert chunks.numel() >= 2 * n_chunks and seq_chunk0.numel() >= n_seqs + 1
+    if freq is not None:
+        _need(freq, "freq", torch.float32)
+        _need(positions, "positions", torch.int32)
+        assert freq.numel() >= rot // 2 and positions.numel() >= n
+    else:
+        rot = 0
+    scratch = torch.empty(n_chunks * n_heads * dim * vdim, dtype=torch.float32, device=proj.device)
+    check(library().mx_retention_chunked(_ptr(proj), proj.stride(0), q_col, k_col, v_col, g_col, _ptr(head_decay),
+                                         float(q_scale), float(eps), _ptr(positions) if freq is not None else None,
+                                         _ptr(freq), int(rot), _ptr(state), _ptr(cu_q), _ptr(state_slots), n_seqs,
+                                         _ptr(chunks), _ptr(seq_chunk0), n_chunks, _ptr(scratch), _ptr(out),
+                                         dtype_code(out.dtype), out.stride(0), n_heads, dim, vdim, _stream()),
+          "retention_chunked")
+    _launched(3)
+
+
 # ---------------------------------------------------------------------- short convolutions, selective recurrence
 def conv_norm_kv_write(proj: torch.Tensor, bias: torch.Tensor | None, conv: torch.Tensor, q_weight: torch.Tensor,
                        k_weight: torch.Tensor | None, eps: float, temperature: tuple[float, float], state: torch.Tensor | None,
@@ -1583,20 +1621,32 @@ def _scan_operands(u, low, dt_bias, a_log2, d, z, state, state_offset, out, n_st
 def selective_scan(u: torch.Tensor, raw: torch.Tensor, low: torch.Tensor, dt_bias: torch.Tensor, a_log2: torch.Tensor,
                    d: torch.Tensor, z: torch.Tensor, state: torch.Tensor, state_offset: int, cu_q: torch.Tensor,
                    state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor, n_states: int, dt_rank: int,
-                   out_scale: float = 1.0) -> None:
+                   out_scale: float = 1.0, chunked: tuple | None = None) -> None:
     """Every sequence's tokens in order, from and to the recurrent part of its ``state`` vector ([channels, n_states] at
     ``state_offset``): ``dt = softplus(raw + dt_bias)``, ``S <- exp(dt A) S + dt u B``,
     ``out = (S C + d u) * silu(z) * out_scale``. ``raw`` float32 [tokens, channels]; ``low`` float32 rows
-    ``[dt_rank | B | C]``; ``a_log2`` is A * log2(e); ``u`` and ``out`` in the activation dtype, ``z`` in it or float32."""
+    ``[dt_rank | B | C]``; ``a_log2`` is A * log2(e); ``u`` and ``out`` in the activation dtype, ``z`` in it or float32.
+    ``chunked`` = (chunks, seq_chunk0, n_chunks, chunk tokens): ``scan_chunk_lists`` on the device, for long portions of few
+    sequences; the chunks run in parallel (three launches)."""
     n, channels = _scan_operands(u, low, dt_bias, a_log2, d, z, state, state_offset, out, n_states, dt_rank)
     _need(raw, "raw", torch.float32)
     assert tuple(raw.shape) == (n, channels)
-    check(library().mx_selective_scan(_ptr(u), _ptr(raw), raw.stride(0), _ptr(low), low.stride(0), _ptr(dt_bias),
-                                      _ptr(a_log2), _ptr(d), _ptr(z), dtype_code(z.dtype), z.stride(0), _ptr(state),
-                                      state.stride(0), int(state_offset), _ptr(cu_q), _ptr(state_slots), _ptr(out),
-                                      dtype_code(out.dtype), out.stride(0), n_seqs, channels, n_states, dt_rank,
-                                      float(out_scale), _stream()), "selective_scan")
-    _launched()
+    arguments = (_ptr(u), _ptr(raw), raw.stride(0), _ptr(low), low.stride(0), _ptr(dt_bias), _ptr(a_log2), _ptr(d), _ptr(z),
+                 dtype_code(z.dtype), z.stride(0), _ptr(state), state.stride(0), int(state_offset), _ptr(cu_q),
+                 _ptr(state_slots), _ptr(out), dtype_code(out.dtype), out.stride(0), n_seqs, channels, n_states, dt_rank,
+                 float(out_scale))
+    if chunked is None:
+        check(library().mx_selective_scan(*arguments, _stream()), "selective_scan")
+        _launched()
+        return
+    chunks, first, n_chunks, size = chunked
+    _need(chunks, "chunks", torch.int32)
+    _need(first, "seq_chunk0", torch.int32)
+    assert chunks.numel() >= 2 * n_chunks and first.numel() >= n_seqs + 1
+    scratch = torch.empty(n_chunks * channels * (n_states + 1), dtype=torch.float32, device=u.device)
+    check(library().mx_selective_scan_chunked(*arguments, _ptr(chunks), _ptr(first), n_chunks, size, _ptr(scratch), _stream()),
+          "selective_scan_chunked")
+    _launched(3)
 
 
 def selective_step(u: torch.Tensor, low: torch.Tensor, dt_weight: torch.Tensor, dt_bias: torch.Tensor,

@@ -67,11 +67,14 @@ _SIGNATURES: dict[str, tuple[list, object]] = {
     "mx_gla_decay": ([P, I, P, P, F, P, I, I, I, P], I),
     "mx_gla_scan": ([P, I, I, I, I, P, F, P, P, P, P, I, I, I, I, P], I),
     "mx_retention_scan": ([P, I, I, I, I, P, F, P, P, P, P, I, I, I, I, P, P, I, P], I),
+    "mx_retention_chunk_tokens": ([], I),
+    "mx_retention_chunked": ([P, I, I, I, I, I, P, F, F, P, P, I, P, P, P, I, P, P, I, P, P, I, I, I, I, I, P], I),
     "mx_rotate_heads": ([P, I, I, I, I, I, I, P, P, P], I),
     "mx_conv_norm_kv_write": ([P, I, P, P, I, P, P, F, F, F, P, L, P, P, P, P, P, P, L, I, P, I, I, I, I, I, I, I, I, P, P], I),
     "mx_conv_state_update": ([P, I, I, P, P, L, P, P, I, I, I, P], I),
     "mx_conv_silu": ([P, I, I, P, P, P, L, P, P, P, P, I, I, I, I, P], I),
     "mx_selective_scan": ([P, P, I, P, I, P, P, P, P, I, I, P, L, L, P, P, P, I, I, I, I, I, I, F, P], I),
+    "mx_selective_scan_chunked": ([P, P, I, P, I, P, P, P, P, I, I, P, L, L, P, P, P, I, I, I, I, I, I, F, P, P, I, I, P, P], I),
     "mx_selective_step": ([P, P, I, P, P, P, P, P, I, I, P, L, L, P, P, P, I, I, I, I, I, I, F, P], I),
     "mx_gla_norm_gate": ([P, P, I, P, F, P, I, I, I, I, P], I),
     "mx_moe_route": ([P, I, I, P, I, I, I, I, I, F, I, P, P, P, P, I, P], I),

@@ -13,8 +13,9 @@ and the gate are float in both dtypes; only the large projections run in the run
 
 Retention (``RetentionSpec``) decays by one constant per head: ``S_t = decay_h S_(t-1) + k_t v_t^T``, ``o_t = S_t^T q_t`` with
 q and k rotated over their first entries. It shares the recurrence's kernel (which takes no decay operand then), the
-state's layout and the kernel behind it (no weight in its norm). Long portions are rotated by a pass of their own, steps
-of one token a sequence on the operands' way into the recurrence.
+state's layout and the kernel behind it (no weight in its norm); short portions are rotated by a pass of their own, steps
+of one token a sequence on the operands' way into the recurrence. Long portions of heads of up to 128 x 128 run in chunks
+of tokens whose products take the place of the updates, with rotation, norm and gate in the same kernels.
 """
 
 from __future__ import annotations
@@ -131,6 +132,22 @@ class Retention(BranchMixer):
         rotation = {}
         if self.position is not None:
             freq, rot = self.position.frequencies, s.position.rotary_dim
+        if not one_token_each(ctx) and max(s.head_dim, s.value_dim) <= 128 and \
+                max(ctx.host.q_lens) > kernels.retention_chunk_tokens() // 2:
+            # long portions in chunks of tokens, products in place of updates
+            size = kernels.retention_chunk_tokens()
+            key = ("retention_chunks", size)
+            if key not in ctx.memo:
+                chunks, first = kernels.scan_chunk_lists(ctx.host.q_lens, size)
+                both = torch.tensor(chunks + first, dtype=torch.int32).to(proj.device, non_blocking=True)
+                ctx.memo[key] = (both[:len(chunks)], both[len(chunks):], len(chunks) // 2)
+            if self.position is not None:
+                rotation = {"positions": ctx.positions, "freq": freq, "rot": rot}
+            kernels.retention_chunked(proj, 0, keys, 2 * keys, 2 * keys + values, self.decay, s.key_scale, s.eps,
+                                      binding.state, ctx.cu_q, ctx.state_slots, ctx.n_seqs, *ctx.memo[key], out,
+                                      s.num_heads, s.head_dim, s.value_dim, **rotation)
+            return
+        if self.position is not None:
             if one_token_each(ctx):
                 rotation = {"positions": ctx.positions, "freq": freq, "rot": rot}
             else:                                                     # q and k heads lie side by side

@@ -24,6 +24,12 @@ from matricxon_b200.parts.base import BranchMixer, StateRequest, register_part
 from matricxon_b200.weights.loader import WeightSpec
 
 
+# tokens per chunk of a long portion, and the channels (over all sequences) per SM from which on the token-by-token walk
+# has warps enough
+CHUNK_TOKENS = 128
+CHANNELS_THAT_FILL = 96
+
+
 @register_part("mixer", "selective_scan")
 class SelectiveScan(BranchMixer):
     capturable = True
@@ -79,5 +85,14 @@ class SelectiveScan(BranchMixer):
             kernels.cast_columns(rank_rows, rounded)
             rank_rows = rounded
         raw = linear(rank_rows, self.dt_weight, None, EPILOGUE_F32, backend=rt.gemm_backend)
+        chunked = None
+        if ctx.n_seqs * c < CHANNELS_THAT_FILL * ctx.sm_count and max(ctx.host.q_lens) > 2 * CHUNK_TOKENS:
+            # a long portion of few sequences: token by token it would be left to a few warps per SM
+            key = ("selective_chunks", CHUNK_TOKENS)
+            if key not in ctx.memo:
+                chunks, first = kernels.scan_chunk_lists(ctx.host.q_lens, CHUNK_TOKENS)
+                both = torch.tensor(chunks + first, dtype=torch.int32).to(proj.device, non_blocking=True)
+                ctx.memo[key] = (both[:len(chunks)], both[len(chunks):], len(chunks) // 2, CHUNK_TOKENS)
+            chunked = ctx.memo[key]
         kernels.selective_scan(u, raw, low, self.dt_bias, self.a_log2, self.d, z, state, recurrent, ctx.cu_q,
-                               ctx.state_slots, ctx.n_seqs, out, s.states, s.dt_rank, scale)
+                               ctx.state_slots, ctx.n_seqs, out, s.states, s.dt_rank, scale, chunked=chunked)

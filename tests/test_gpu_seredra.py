@@ -559,6 +559,75 @@ def test_retention_kernels(heads, dim, vdim, rot):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("heads, dim, vdim, rot", [(3, 20, 28, 12), (2, 64, 128, 64), (4, 128, 64, 128), (1, 96, 24, 2),
+                                                   (5, 13, 7, 6), (2, 128, 128, 0), (3, 64, 64, 32)])
+def test_retention_in_chunks(dtype, heads, dim, vdim, rot):
+    """Long and short portions in one launch (whole chunks, one token more and less, single tokens), the norm and the gate
+    in the same kernels, from and to the slots, against the plain recurrence over the whole sequences."""
+    gen = torch.Generator().manual_seed(dim + rot)
+    decay = torch.tensor([0.0, 1.0, 0.97, 0.5, 0.9])[-heads:]
+    cuts, slots = [[64, 1, 130], [63, 65, 64], [200, 128, 1], [0, 1, 7]], [3, 0, 2, 1]
+    width = heads * (2 * dim + 2 * vdim)
+    rows_of = [torch.randn(sum(c), width, generator=gen) for c in cuts]
+    spec, freq = (turned(rot, 400.0), plain.frequencies(rot, 400.0)[0].float().to(DEVICE)) if rot else (None, None)
+    state = torch.zeros(4, heads, dim, vdim, device=DEVICE)
+    size, eps = kernels.retention_chunk_tokens(), 1e-4
+    done, got = [0] * len(cuts), [[] for _ in cuts]
+    for live, batch in batches_of(cuts, slots):
+        rows = torch.cat([rows_of[s][done[s]:done[s] + k] for s, k in zip(live, batch.q_lens)])
+        proj = torch.cat([rows, torch.full((batch.n, 4), 9.0)], 1).to(DEVICE)
+        chunks, first = kernels.scan_chunk_lists(batch.q_lens, size)
+        wide = torch.zeros(batch.n, heads * vdim + 16, dtype=dtype, device=DEVICE)
+        rotation = dict(positions=batch.positions, freq=freq, rot=rot) if rot else {}
+        kernels.retention_chunked(proj, 0, heads * dim, 2 * heads * dim, heads * (2 * dim + vdim), decay.to(DEVICE),
+                                  dim ** -0.5, eps, state, batch.cu_q, batch.slots, len(live), ints(chunks), ints(first),
+                                  len(chunks) // 2, wide[:, 8:8 + heads * vdim], heads, dim, vdim, **rotation)
+        assert float(wide[:, :8].abs().max()) == 0.0 and float(wide[:, 8 + heads * vdim:].abs().max()) == 0.0
+        for i, s in enumerate(live):
+            got[s].append(wide[batch.rows(i), 8:8 + heads * vdim].double().cpu())
+            done[s] += batch.q_lens[i]
+    tol = 2e-4 if dtype == torch.float32 else 1e-2
+    for s, rows in enumerate(rows_of):
+        p64, pos = rows.double(), torch.arange(len(rows))
+        q = plain.rotate(p64[:, :heads * dim].view(-1, heads, dim), pos, spec)
+        k = plain.rotate(p64[:, heads * dim:2 * heads * dim].view(-1, heads, dim), pos, spec) * dim ** -0.5
+        v = p64[:, 2 * heads * dim:heads * (2 * dim + vdim)].view(-1, heads, vdim)
+        o = plain.linear_recurrence(q, k, v, decay.double())
+        want = plain.unit(o, eps).reshape(len(rows), -1) * plain.silu(p64[:, heads * (2 * dim + vdim):])
+        mine = torch.cat(got[s])
+        # a head whose o is nearly zero for all its values is ill-conditioned under its own norm: rounding shows there
+        hard = (o.pow(2).mean(-1).sqrt() < 1e-2)[:, :, None].expand(-1, -1, vdim).reshape(len(rows), -1)
+        error = ((mine - want).abs() / (want.abs() + 1.0)).masked_fill(hard, 0.0)
+        assert float(error.max()) < tol, (s, float(error.max()))
+        assert float(hard.double().mean()) < 0.05
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("channels, n, rank, size", [(72, 13, 9, 32), (160, 16, 8, 128), (33, 100, 5, 7), (40, 1, 3, 50)])
+def test_selective_recurrence_in_chunks(dtype, channels, n, rank, size):
+    """The three-launch form beside the walk it replaces, over several steps and unequal portions, from and to the slots."""
+    gen = torch.Generator().manual_seed(channels * n)
+    dt_bias, d = torch.rand(channels, generator=gen) * 5 - 4, torch.randn(channels, generator=gen)
+    a_log2 = -torch.exp(torch.rand(channels, n, generator=gen) * 4 - 2)
+    constants = dt_bias.to(DEVICE), a_log2.to(DEVICE), d.to(DEVICE)
+    state = torch.randn(4, 24 + channels * n, generator=gen).to(DEVICE)
+    whole = state.clone()
+    for q_lens in ([300, 1, size, 64], [2, size + 1, 90], [1, 1, 1, 3 * size]):
+        batch = Batch(q_lens, [0] * len(q_lens), [2, 0, 3, 1][:len(q_lens)])
+        u, z = (torch.randn(batch.n, channels, generator=gen).to(dtype).to(DEVICE) for _ in range(2))
+        raw, low = torch.randn(batch.n, channels, generator=gen).to(DEVICE), torch.randn(batch.n, rank + 2 * n, generator=gen).to(DEVICE)
+        chunks, first = kernels.scan_chunk_lists(q_lens, size)
+        outs = []
+        for kept, chunked in ((whole, None), (state, (ints(chunks), ints(first), len(chunks) // 2, size))):
+            out = torch.empty(batch.n, channels, dtype=dtype, device=DEVICE)
+            kernels.selective_scan(u, raw, low, *constants, z, kept, 24, batch.cu_q, batch.slots, len(q_lens), out, n, rank,
+                                   0.7, chunked=chunked)
+            outs.append(out.double())
+        tol = 1e-4 if dtype == torch.float32 else 1e-2
+        assert torch.allclose(*outs, rtol=tol, atol=tol) and torch.allclose(state, whole, rtol=1e-4, atol=1e-4)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("heads, vdim", [(3, 28), (2, 128), (1, 300)])
 def test_heads_normalised_without_a_weight_and_gated(dtype, heads, vdim):
     gen = torch.Generator().manual_seed(vdim)
