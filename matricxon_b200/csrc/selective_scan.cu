@@ -302,11 +302,24 @@ selective_carry_kernel(const ScanParams p) {
     const float a = p.a_log2[i];
     float s = p.state[(size_t)p.state_slots[seq] * p.state_stride + p.state_offset + i];
     const int end = p.seq_chunk0[seq + 1];
-    for (int chunk = p.seq_chunk0[seq]; chunk < end; ++chunk) {
-        float* here = p.chunk_state + (size_t)chunk * p.channels * p.n + i;
-        const float reached = chunk + 1 < end ? *here : 0.f;
-        *here = s;
-        if (chunk + 1 < end) s = fmaf(exp2_fast(p.chunk_dt[(size_t)chunk * p.channels + c] * a), s, reached);
+    const size_t stride = (size_t)p.channels * p.n;
+    constexpr int AHEAD = 8;                                 // a group's maps are read before its first start is written
+    for (int chunk = p.seq_chunk0[seq]; chunk < end; chunk += AHEAD) {
+        float* here = p.chunk_state + (size_t)chunk * stride + i;
+        const float* dt = p.chunk_dt + (size_t)chunk * p.channels + c;
+        float reached[AHEAD], passed[AHEAD];
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g) {
+            const bool maps = chunk + g + 1 < end;           // the last chunk hands nothing on
+            reached[g] = maps ? here[g * stride] : 0.f;
+            passed[g] = maps ? dt[(size_t)g * p.channels] : 0.f;
+        }
+#pragma unroll
+        for (int g = 0; g < AHEAD; ++g) {
+            if (chunk + g >= end) break;
+            here[g * stride] = s;
+            s = fmaf(exp2_fast(passed[g] * a), s, reached[g]);
+        }
     }
 }
 

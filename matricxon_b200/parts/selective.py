@@ -26,7 +26,7 @@ from matricxon_b200.weights.loader import WeightSpec
 
 # tokens per chunk of a long portion, and the channels (over all sequences) per SM from which on the token-by-token walk
 # has warps enough
-CHUNK_TOKENS = 128
+CHUNK_TOKENS = 64
 CHANNELS_THAT_FILL = 96
 
 
