@@ -133,6 +133,14 @@ def _register_builtin() -> None:
         config_class=SeredraConfig,
         build_model=_build_decoder,
     ))
+    from matricxon_b200.config.palelix import PalelixConfig
+
+    register_architecture(ArchitectureEntry(
+        name="Palelix",
+        aliases=("palelix",),
+        config_class=PalelixConfig,
+        build_model=_build_decoder,
+    ))
 
 
 _register_builtin()

@@ -21,7 +21,10 @@
 //   position * freq[i] in float), for portions so short that rotating once per piece of 16 value columns costs less
 //   than a pass of its own. mx_rotate_heads is that pass: heads of float rows rotated in place.
 // mx_gla_norm_gate: out[t][h][e] = o[t][h][e] / sqrt(mean_e(o^2) + eps) * weight[e] * silu(gate[t][h][e]): the
-//   per-head RMS norm (`weight` null: no weight) and the output gate, rounded once.
+//   per-head RMS norm (`weight` null: no weight) and the output gate, rounded once. `sigmoid_gate`: sigmoid in silu's place;
+//   rows of `out` may be `out_ld` apart, the result is multiplied by `out_scale`, and a mean divides by `true_vdim` (heads
+//   filled up with zeros).
+// mx_norm_gate_rows: the same with one norm over a whole row (all heads) and a weight of a row's width, a block per token.
 #include <math.h>
 
 #include "common.cuh"
@@ -93,7 +96,7 @@ gla_decay_kernel(const float* __restrict__ low, int low_ld, const float* __restr
 
 // GLA_SLICES threads share a pair of columns, each with ROWS of the key channels (dim <= GLA_SLICES * ROWS);
 // GLA_TOKENS tokens are staged per round
-template <int ROWS, int GLA_SLICES, int GLA_TOKENS, bool HEAD_DECAY, bool ROTATE>
+template <int ROWS, int GLA_SLICES, int GLA_TOKENS, bool HEAD_DECAY, bool ROTATE, bool SILU>
 __global__ void __launch_bounds__(GLA_COLS / 2 * GLA_SLICES)
 gla_scan_kernel(const float* proj, int ld, int q_col, int k_col, int v_col, const float* decay, float q_scale,
                 float* __restrict__ state, const int* __restrict__ cu_q, const int* __restrict__ state_slots,
@@ -150,6 +153,10 @@ gla_scan_kernel(const float* proj, int ld, int q_col, int k_col, int v_col, cons
             const float* row = proj + (size_t)(base + j) * ld + head * dim + i;
             q_r[u] = live ? row[q_col] : 0.f;
             k_r[u] = live ? row[k_col] : 0.f;
+            if (SILU) {
+                q_r[u] = silu_of<float>(q_r[u]);
+                k_r[u] = silu_of<float>(k_r[u]);
+            }
             if (!HEAD_DECAY) a_r[u] = live ? decay[((size_t)(base + j) * n_heads + head) * dim + i] : 0.f;
             if (ROTATE && live && i < rot) {
                 const int half = rot >> 1, pair = i < half ? i : i - half, away = i < half ? half : -half;
@@ -165,6 +172,7 @@ gla_scan_kernel(const float* proj, int ld, int q_col, int k_col, int v_col, cons
             const int item = tid + u * GLA_THREADS, j = item / GLA_COLS, c = item % GLA_COLS;
             v_r[u] = (item < GLA_TOKENS * GLA_COLS && j < n_here && col0 + c < vdim)
                          ? proj[(size_t)(base + j) * ld + v_col + head * vdim + col0 + c] : 0.f;
+            if (SILU) v_r[u] = silu_of<float>(v_r[u]);
         }
     };
     // one token's operands of this thread, from shared memory into registers (asked for one token ahead)
@@ -251,8 +259,8 @@ gla_scan_kernel(const float* proj, int ld, int q_col, int k_col, int v_col, cons
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-gla_norm_gate_kernel(const float* o, const float* gate, int gate_ld,
-                     const float* __restrict__ weight, float eps, T* __restrict__ out, int n_heads, int vdim) {
+gla_norm_gate_kernel(const float* o, const float* gate, int gate_ld, const float* __restrict__ weight, float eps,
+                     T* __restrict__ out, int n_heads, int vdim, int sigmoid_gate, int out_ld, float out_scale, int true_vdim) {
     pdl_trigger();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     const int h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -274,16 +282,54 @@ gla_norm_gate_kernel(const float* o, const float* gate, int gate_ld,
 #pragma unroll
     for (int u = 0; u < KEPT; ++u) s = fmaf(val[u], val[u], s);
     for (int e = lane + 32 * KEPT; e < vdim; e += 32) s = fmaf(src[e], src[e], s);
-    const float inv = 1.0f / sqrtf(warp_sum(s) / (float)vdim + eps);
+    const float inv = out_scale / sqrtf(warp_sum(s) / (float)true_vdim + eps);
+    T* dst = out + (size_t)t * out_ld + h * vdim;
 #pragma unroll
     for (int u = 0; u < KEPT; ++u) {
         const int e = lane + 32 * u;
         if (e < vdim)
-            out[((size_t)t * n_heads + h) * vdim + e] = from_float<T>(val[u] * inv * (weight ? weight[e] : 1.f) * (g[u] / (1.0f + expf(-g[u]))));
+            dst[e] = from_float<T>(val[u] * inv * (weight ? weight[e] : 1.f) * ((sigmoid_gate ? 1.f : g[u]) / (1.0f + expf(-g[u]))));
     }
     for (int e = lane + 32 * KEPT; e < vdim; e += 32) {
         const float gv = g_row[e];
-        out[((size_t)t * n_heads + h) * vdim + e] = from_float<T>(src[e] * inv * (weight ? weight[e] : 1.f) * (gv / (1.0f + expf(-gv))));
+        dst[e] = from_float<T>(src[e] * inv * (weight ? weight[e] : 1.f) * ((sigmoid_gate ? 1.f : gv) / (1.0f + expf(-gv))));
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+norm_gate_rows_kernel(const float* o, const float* gate, int gate_ld, const float* __restrict__ weight, float eps,
+                      T* __restrict__ out, int width, int sigmoid_gate, int out_ld) {
+    __shared__ float scratch[32];
+    pdl_trigger();
+    constexpr int KEPT = 8;                       // up to 2,048 entries of a row stay in registers
+    const int t = blockIdx.x, tid = threadIdx.x;
+    float w[KEPT], val[KEPT], g[KEPT];
+#pragma unroll
+    for (int u = 0; u < KEPT; ++u) w[u] = weight && tid + 256 * u < width ? weight[tid + 256 * u] : 1.f;
+    pdl_wait();
+    const float* src = after_wait(o) + (size_t)t * width;
+    const float* g_row = after_wait(gate) + (size_t)t * gate_ld;
+    float s = 0.f;
+#pragma unroll
+    for (int u = 0; u < KEPT; ++u) {
+        const int e = tid + 256 * u;
+        val[u] = e < width ? src[e] : 0.f;
+        g[u] = e < width ? g_row[e] : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < KEPT; ++u) s = fmaf(val[u], val[u], s);
+    for (int e = tid + 256 * KEPT; e < width; e += 256) s = fmaf(src[e], src[e], s);
+    const float inv = 1.0f / sqrtf(block_sum(s, scratch) / (float)width + eps);
+    T* dst = out + (size_t)t * out_ld;
+#pragma unroll
+    for (int u = 0; u < KEPT; ++u) {
+        const int e = tid + 256 * u;
+        if (e < width) dst[e] = from_float<T>(val[u] * inv * w[u] * ((sigmoid_gate ? 1.f : g[u]) / (1.0f + expf(-g[u]))));
+    }
+    for (int e = tid + 256 * KEPT; e < width; e += 256) {
+        const float gv = g_row[e];
+        dst[e] = from_float<T>(src[e] * inv * (weight ? weight[e] : 1.f) * ((sigmoid_gate ? 1.f : gv) / (1.0f + expf(-gv))));
     }
 }
 
@@ -306,13 +352,13 @@ __global__ void rotate_heads_kernel(float* rows, int ld, int col, int n_heads, i
     }
 }
 
-template <bool HEAD_DECAY, bool ROTATE>
+template <bool HEAD_DECAY, bool ROTATE, bool SILU>
 void launch_gla_scan(const float* proj, int ld, int q_col, int k_col, int v_col, const float* decay, float q_scale,
                      float* state, const int* cu_q, const int* state_slots, float* out, int n_seqs, int n_heads, int dim,
                      int vdim, const int* positions, const float* freq, int rot, cudaStream_t stream) {
     const dim3 grid(n_seqs, n_heads, (vdim + GLA_COLS - 1) / GLA_COLS);
 #define MX_GLA(ROWS, SLICES, TOKENS)                                                                                  \
-    mx_launch_chained(gla_scan_kernel<ROWS, SLICES, TOKENS, HEAD_DECAY, ROTATE>, grid, dim3(GLA_COLS / 2 * SLICES), 0, \
+    mx_launch_chained(gla_scan_kernel<ROWS, SLICES, TOKENS, HEAD_DECAY, ROTATE, SILU>, grid, dim3(GLA_COLS / 2 * SLICES), 0, \
                       stream, proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q, state_slots, out, n_heads,  \
                       dim, vdim, positions, freq, rot)
     if (dim <= 64) MX_GLA(4, 16, 16);
@@ -341,26 +387,31 @@ extern "C" int mx_gla_scan(const float* proj, int ld, int q_col, int k_col, int 
     if (n_seqs <= 0) return MX_OK;
     if (dim <= 0 || dim > 256) MX_REFUSE("gated linear attention: %d key channels per head (1..256)", dim);
     if (n_heads > 65535 || vdim > 65535 * GLA_COLS) MX_REFUSE("gated linear attention: %d heads of %d values exceed the grid", n_heads, vdim);
-    launch_gla_scan<false, false>(proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q, state_slots, out, n_seqs,
+    launch_gla_scan<false, false, false>(proj, ld, q_col, k_col, v_col, decay, q_scale, state, cu_q, state_slots, out, n_seqs,
                                   n_heads, dim, vdim, nullptr, nullptr, 0, stream);
     return mx_launch_status();
 }
 
 // `head_decay` [n_heads]: S_t = head_decay_h S_(t-1) + k_t v_t^T. `freq` null: q and k are taken as they are, else they
-// are rotated over their first `rot` entries on their way in.
+// are rotated over their first `rot` entries on their way in. `silu`: q, k and v are the silu of what the rows hold (heads
+// that are not rotated).
 extern "C" int mx_retention_scan(const float* proj, int ld, int q_col, int k_col, int v_col, const float* head_decay,
                                  float q_scale, float* state, const int* cu_q, const int* state_slots, float* out,
                                  int n_seqs, int n_heads, int dim, int vdim, const int* positions, const float* freq,
-                                 int rot, cudaStream_t stream) {
+                                 int rot, int silu, cudaStream_t stream) {
     if (n_seqs <= 0) return MX_OK;
     if (dim <= 0 || dim > 256) MX_REFUSE("retention: %d key channels per head (1..256)", dim);
     if (n_heads > 65535 || vdim > 65535 * GLA_COLS) MX_REFUSE("retention: %d heads of %d values exceed the grid", n_heads, vdim);
     if (rot < 0 || rot % 2 != 0 || rot > dim) MX_REFUSE("retention: %d rotated entries in a head of %d", rot, dim);
-    if (freq != nullptr && rot > 0)
-        launch_gla_scan<true, true>(proj, ld, q_col, k_col, v_col, head_decay, q_scale, state, cu_q, state_slots, out,
+    if (silu && freq != nullptr && rot > 0) MX_REFUSE("retention: activated heads of %d entries are not rotated", dim);
+    if (silu)
+        launch_gla_scan<true, false, true>(proj, ld, q_col, k_col, v_col, head_decay, q_scale, state, cu_q, state_slots, out,
+                                           n_seqs, n_heads, dim, vdim, nullptr, nullptr, 0, stream);
+    else if (freq != nullptr && rot > 0)
+        launch_gla_scan<true, true, false>(proj, ld, q_col, k_col, v_col, head_decay, q_scale, state, cu_q, state_slots, out,
                                     n_seqs, n_heads, dim, vdim, positions, freq, rot, stream);
     else
-        launch_gla_scan<true, false>(proj, ld, q_col, k_col, v_col, head_decay, q_scale, state, cu_q, state_slots, out,
+        launch_gla_scan<true, false, false>(proj, ld, q_col, k_col, v_col, head_decay, q_scale, state, cu_q, state_slots, out,
                                      n_seqs, n_heads, dim, vdim, nullptr, nullptr, 0, stream);
     return mx_launch_status();
 }
@@ -379,14 +430,30 @@ extern "C" int mx_rotate_heads(float* rows, int ld, int col, int n_tokens, int n
 }
 
 extern "C" int mx_gla_norm_gate(const float* o, const float* gate, int gate_ld, const float* weight, float eps, void* out,
-                                int dtype, int n_tokens, int n_heads, int vdim, cudaStream_t stream) {
+                                int dtype, int n_tokens, int n_heads, int vdim, int sigmoid_gate, int out_ld, float out_scale,
+                                int true_vdim, cudaStream_t stream) {
     if (n_tokens <= 0) return MX_OK;
+    if (out_ld < n_heads * vdim || true_vdim <= 0 || true_vdim > vdim) MX_REFUSE("norm and gate: %d values of %d in rows of %d", true_vdim, vdim, out_ld);
     const dim3 grid(n_tokens, (n_heads + 3) / 4);
     if (dtype == MX_DTYPE_F32)
         mx_launch_chained(gla_norm_gate_kernel<float>, grid, dim3(128), 0, stream, o, gate, gate_ld, weight, eps,
-                          (float*)out, n_heads, vdim);
+                          (float*)out, n_heads, vdim, sigmoid_gate, out_ld, out_scale, true_vdim);
     else
         mx_launch_chained(gla_norm_gate_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, o, gate, gate_ld, weight, eps,
-                          (__nv_bfloat16*)out, n_heads, vdim);
+                          (__nv_bfloat16*)out, n_heads, vdim, sigmoid_gate, out_ld, out_scale, true_vdim);
+    return mx_launch_status();
+}
+
+// out[t][e] = o[t][e] / sqrt(mean_e(o^2) + eps) * weight[e] * act(gate[t][e]) over rows of `width` entries, act silu or sigmoid
+extern "C" int mx_norm_gate_rows(const float* o, const float* gate, int gate_ld, const float* weight, float eps, void* out,
+                                 int dtype, int n_tokens, int width, int sigmoid_gate, int out_ld, cudaStream_t stream) {
+    if (n_tokens <= 0) return MX_OK;
+    if (width <= 0 || out_ld < width) MX_REFUSE("norm and gate: rows of %d entries in rows of %d", width, out_ld);
+    if (dtype == MX_DTYPE_F32)
+        mx_launch_chained(norm_gate_rows_kernel<float>, dim3(n_tokens), dim3(256), 0, stream, o, gate, gate_ld, weight, eps,
+                          (float*)out, width, sigmoid_gate, out_ld);
+    else
+        mx_launch_chained(norm_gate_rows_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(256), 0, stream, o, gate, gate_ld, weight,
+                          eps, (__nv_bfloat16*)out, width, sigmoid_gate, out_ld);
     return mx_launch_status();
 }

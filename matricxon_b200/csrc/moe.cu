@@ -11,7 +11,8 @@
 // mx_moe_route_softmax: the same outputs from another rule. The router has `n_experts + n_identity` rows; the scores
 //   are the softmax over all of them (of logit + bias[e] where a bias is given: with it and no correction the rule is
 //   "the `top` largest logits, weighted by the softmax over those alone"); the choice ranks score + correction[e] (a float per row, optional) and takes the
-//   `top` largest (ties to the lower index); the weights are the winners' plain scores over their sum (+ 1e-20). The
+//   `top` largest (ties to the lower index); the weights are the winners' plain scores over their sum (+ 1e-20). With
+//   `n_groups` > 1 only rows of the `keep` runs of neighbours whose best score is largest may be chosen. The
 //   last `n_identity` rows stand for experts without matrices that return their input: such a pair keeps its id
 //   (>= n_experts), is counted nowhere and gets no sorted row; the combine kernels add weight * input for it.
 // mx_moe_plan (one block): from the counts, the first sorted row of every expert and the list of row tiles
@@ -167,7 +168,7 @@ moe_route_kernel(const T* __restrict__ h, int ld, const float* __restrict__ rout
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_route_softmax_kernel(const T* __restrict__ h, int ld, const float* __restrict__ router, int K, int n_experts,
-                         int n_identity, int top, const float* __restrict__ correction,
+                         int n_identity, int top, int n_groups, int keep, const float* __restrict__ correction,
                          const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights,
                          int* __restrict__ counts, int* __restrict__ place) {
     extern __shared__ __align__(16) float route_s[];
@@ -175,6 +176,7 @@ moe_route_softmax_kernel(const T* __restrict__ h, int ld, const float* __restric
     float* h_s = route_s;                         // [K]
     float* score = h_s + K;                       // [rows]: logits, then softmax scores
     float* open = score + n_rows;                 // [rows]: score + correction while the row may still be chosen
+    float* worth = open + n_rows;                 // [groups]
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     router_logits(h + (size_t)t * ld, router, K, n_rows, h_s, score);
     if (threadIdx.x >= 32) return;
@@ -197,6 +199,29 @@ moe_route_softmax_kernel(const T* __restrict__ h, int ld, const float* __restric
         open[e] = sc + (correction ? correction[e] : 0.f);
     }
     __syncwarp();
+    if (n_groups > 1 && keep < n_groups) {
+        // a run of neighbours is worth its best score; the rows of all but the best runs are closed
+        const int per = n_rows / n_groups;
+        for (int g = lane; g < n_groups; g += 32) {
+            float best = open[g * per];
+            for (int e = g * per + 1; e < (g + 1) * per; ++e) best = fmaxf(best, open[e]);
+            worth[g] = best;
+        }
+        __syncwarp();
+        for (int round = 0; round < keep; ++round) {
+            float v = -1.f;                       // scores are not negative; a run that is kept gets -2
+            int i = 0x7fffffff;
+            for (int g = lane; g < n_groups; g += 32)
+                if (worth[g] > v) { v = worth[g]; i = g; }
+            arg_best(v, i);
+            __syncwarp();
+            if (lane == 0 && i < n_groups) worth[i] = -2.f;
+            __syncwarp();
+        }
+        for (int e = lane; e < n_rows; e += 32)
+            if (worth[e / per] != -2.f) open[e] = -INFINITY;
+        __syncwarp();
+    }
     float total = 0.f;
     for (int slot = 0; slot < top; ++slot) {
         float v = -INFINITY;
@@ -487,22 +512,25 @@ extern "C" int mx_moe_route(const void* h, int dtype, int ld, const float* route
 }
 
 extern "C" int mx_moe_route_softmax(const void* h, int dtype, int ld, const float* router, int K, int n_experts,
-                                    int n_identity, int top, const float* correction, const float* bias, int* ids,
-                                    float* weights, int* counts, int* place, int n_tokens, cudaStream_t stream) {
+                                    int n_identity, int top, int n_groups, int keep, const float* correction,
+                                    const float* bias, int* ids, float* weights, int* counts, int* place, int n_tokens,
+                                    cudaStream_t stream) {
     if (n_tokens <= 0) return MX_OK;
     const int n_rows = n_experts + n_identity;
     if (n_experts < 0 || n_identity < 0 || top <= 0 || top > n_rows)
         MX_REFUSE("router: top %d of %d experts and %d without matrices", top, n_experts, n_identity);
-    const size_t smem = ((size_t)K + 2 * (size_t)n_rows) * sizeof(float);
+    if (n_groups <= 0 || n_rows % n_groups || keep <= 0 || keep > n_groups || keep * (n_rows / n_groups) < top)
+        MX_REFUSE("router: %d of %d groups of %d rows cannot supply %d", keep, n_groups, n_rows, top);
+    const size_t smem = ((size_t)K + 2 * (size_t)n_rows + n_groups) * sizeof(float);
     if (smem > 48 * 1024) MX_REFUSE("router: %zu bytes of shared memory for K = %d and %d rows", smem, K, n_rows);
     if (dtype == MX_DTYPE_F32)
         moe_route_softmax_kernel<float><<<n_tokens, 256, smem, stream>>>((const float*)h, ld, router, K, n_experts,
-                                                                        n_identity, top, correction, bias, ids,
+                                                                        n_identity, top, n_groups, keep, correction, bias, ids,
                                                                         weights, counts, place);
     else
         moe_route_softmax_kernel<__nv_bfloat16><<<n_tokens, 256, smem, stream>>>(
-            (const __nv_bfloat16*)h, ld, router, K, n_experts, n_identity, top, correction, bias, ids, weights, counts,
-            place);
+            (const __nv_bfloat16*)h, ld, router, K, n_experts, n_identity, top, n_groups, keep, correction, bias, ids, weights,
+            counts, place);
     return mx_launch_status();
 }
 

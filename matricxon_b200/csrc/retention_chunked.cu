@@ -10,6 +10,7 @@
 // A block holds the chunk's q, k and v rows in shared memory (rotated in place: pairs (i, i + rot/2), angle
 // position * freq[i] in float), and its start state in the keys' place once the scores exist (two blocks an SM); 256 threads own 4 x 8 pieces of the outputs (8 x 8 of a map). Heads of up to 128 key
 // channels and 128 values, padded with zeros to 64 or 128. Rows of tokens that the chunk does not have are skipped.
+// `silu`: q, k and v are the silu of what the projection holds. `raw`: o itself goes out, in float, without norm and gate.
 // Equal to the token-by-token recurrence up to float rounding, however the sequence was cut.
 #include <math.h>
 
@@ -32,12 +33,13 @@ struct RetentionParams {
     float* chunk_state;         // [n_chunks][heads][dim][vdim]: what a chunk adds, then its start state
     int ld, q_col, k_col, v_col, g_col, heads, dim, vdim, rot, out_ld;
     float q_scale, eps;
+    int silu, raw;
     int vec;                    // widths, strides and columns in groups of four
 };
 
 // rows of one head ([tokens][width] at column `col`) into shared memory [RC_TOKENS][P + RC_PAD], zeros beyond `n` and `width`
 template <int P>
-__device__ __forceinline__ void load_rows(float* dst, const float* src, int ld, int n, int width, int vec) {
+__device__ __forceinline__ void load_rows(float* dst, const float* src, int ld, int n, int width, int vec, int silu = 0) {
     constexpr int S = P + RC_PAD;
     if (vec) {
         constexpr int ITEMS = RC_TOKENS * (P / 4) / RC_THREADS;
@@ -51,12 +53,14 @@ __device__ __forceinline__ void load_rows(float* dst, const float* src, int ld, 
 #pragma unroll
         for (int i = 0; i < ITEMS; ++i) {
             const int item = threadIdx.x + i * RC_THREADS, j = item / (P / 4), c = (item % (P / 4)) * 4;
+            if (silu) v[i] = make_float4(silu_of<float>(v[i].x), silu_of<float>(v[i].y), silu_of<float>(v[i].z), silu_of<float>(v[i].w));
             *reinterpret_cast<float4*>(dst + j * S + c) = v[i];
         }
     } else {
         for (int item = threadIdx.x; item < RC_TOKENS * P; item += RC_THREADS) {
             const int j = item / P, c = item % P;
-            dst[j * S + c] = j < n && c < width ? src[(size_t)j * ld + c] : 0.f;
+            const float v = j < n && c < width ? src[(size_t)j * ld + c] : 0.f;
+            dst[j * S + c] = silu ? silu_of<float>(v) : v;
         }
     }
 }
@@ -99,8 +103,8 @@ retention_maps_kernel(const RetentionParams p) {
     const int seq = p.chunks[2 * chunk], t0 = p.cu_q[seq] + p.chunks[2 * chunk + 1];
     const int n = min(RC_TOKENS, p.cu_q[seq + 1] - t0);
     const float* rows = p.proj + (size_t)t0 * p.ld;
-    load_rows<DP>(k_s, rows + p.k_col + head * p.dim, p.ld, n, p.dim, p.vec);
-    load_rows<VP>(v_s, rows + p.v_col + head * p.vdim, p.ld, n, p.vdim, p.vec);
+    load_rows<DP>(k_s, rows + p.k_col + head * p.dim, p.ld, n, p.dim, p.vec, p.silu);
+    load_rows<VP>(v_s, rows + p.v_col + head * p.vdim, p.ld, n, p.vdim, p.vec, p.silu);
     if (tid < RC_TOKENS) power[tid] = powf(p.decay[head], (float)max(n - 1 - tid, 0));
     __syncthreads();
     if (p.freq) {
@@ -203,9 +207,9 @@ retention_outputs_kernel(const RetentionParams p, T* __restrict__ out) {
     const int seq = p.chunks[2 * chunk], t0 = p.cu_q[seq] + p.chunks[2 * chunk + 1];
     const int n = min(RC_TOKENS, p.cu_q[seq + 1] - t0);
     const float* rows = p.proj + (size_t)t0 * p.ld;
-    load_rows<DP>(q_s, rows + p.q_col + head * p.dim, p.ld, n, p.dim, p.vec);
-    load_rows<DP>(k_s, rows + p.k_col + head * p.dim, p.ld, n, p.dim, p.vec);
-    load_rows<VP>(v_s, rows + p.v_col + head * p.vdim, p.ld, n, p.vdim, p.vec);
+    load_rows<DP>(q_s, rows + p.q_col + head * p.dim, p.ld, n, p.dim, p.vec, p.silu);
+    load_rows<DP>(k_s, rows + p.k_col + head * p.dim, p.ld, n, p.dim, p.vec, p.silu);
+    load_rows<VP>(v_s, rows + p.v_col + head * p.vdim, p.ld, n, p.vdim, p.vec, p.silu);
     const float* start = p.chunk_state + ((size_t)chunk * p.heads + head) * p.dim * p.vdim;
     if (tid <= RC_TOKENS) power[tid] = powf(p.decay[head], (float)tid);
     __syncthreads();
@@ -313,6 +317,18 @@ retention_outputs_kernel(const RetentionParams p, T* __restrict__ out) {
         for (int o = 8; o > 0; o >>= 1) squares += __shfl_xor_sync(row_lanes, squares, o);
         const int i = row0 + r;
         if (i >= n) continue;
+        if (p.raw) {
+            T* dst = out + (size_t)(t0 + i) * p.out_ld + (size_t)head * p.vdim;
+#pragma unroll
+            for (int b = 0; b < CB; ++b) {
+                const int e = 4 * tx + 64 * b;
+                const float o[4] = {acc[r][b].x, acc[r][b].y, acc[r][b].z, acc[r][b].w};
+#pragma unroll
+                for (int x = 0; x < 4; ++x)
+                    if (e + x < p.vdim) dst[e + x] = from_float<T>(o[x]);
+            }
+            continue;
+        }
         const float inv = 1.0f / sqrtf(squares / (float)p.vdim + p.eps);
         const float* gate = rows + (size_t)i * p.ld + p.g_col + head * p.vdim;
         T* dst = out + (size_t)(t0 + i) * p.out_ld + (size_t)head * p.vdim;
@@ -368,7 +384,7 @@ extern "C" int mx_retention_chunked(const float* proj, int ld, int q_col, int k_
                                     float q_scale, float eps, const int* positions, const float* freq, int rot, float* state,
                                     const int* cu_q, const int* state_slots, int n_seqs, const int* chunks,
                                     const int* seq_chunk0, int n_chunks, float* scratch, void* out, int dtype, int out_ld,
-                                    int heads, int dim, int vdim, cudaStream_t stream) {
+                                    int heads, int dim, int vdim, int silu, int raw, cudaStream_t stream) {
     if (n_seqs <= 0 || n_chunks <= 0) return MX_OK;
     if (dim <= 0 || dim > 128 || vdim <= 0 || vdim > 128) MX_REFUSE("chunked retention: heads of %d x %d (at most 128 x 128)", dim, vdim);
     if (heads <= 0 || heads > 65535) MX_REFUSE("chunked retention: %d heads exceed the grid", heads);
@@ -377,7 +393,7 @@ extern "C" int mx_retention_chunked(const float* proj, int ld, int q_col, int k_
     p.proj = proj; p.decay = decay; p.positions = positions; p.freq = rot > 0 ? freq : nullptr; p.cu_q = cu_q;
     p.state_slots = state_slots; p.chunks = chunks; p.seq_chunk0 = seq_chunk0; p.state = state; p.chunk_state = scratch;
     p.ld = ld; p.q_col = q_col; p.k_col = k_col; p.v_col = v_col; p.g_col = g_col; p.heads = heads; p.dim = dim; p.vdim = vdim;
-    p.rot = rot; p.out_ld = out_ld; p.q_scale = q_scale; p.eps = eps;
+    p.silu = silu; p.raw = raw; p.rot = rot; p.out_ld = out_ld; p.q_scale = q_scale; p.eps = eps;
     p.vec = (dim | vdim | ld | q_col | k_col | v_col) % 4 == 0 && ((uintptr_t)proj | (uintptr_t)scratch) % 16 == 0;
     if (dtype == MX_DTYPE_F32) return pick_retention<float>(p, (float*)out, n_seqs, n_chunks, stream);
     return pick_retention<__nv_bfloat16>(p, (__nv_bfloat16*)out, n_seqs, n_chunks, stream);

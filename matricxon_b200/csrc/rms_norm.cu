@@ -214,7 +214,8 @@ __global__ void rmsnorm_vec_kernel(const float* x, const int* __restrict__ rows,
     }
 }
 
-// The same behind a residual sum that is still to be formed: the row is x + (acc + col_bias), written back on the way.
+// The same behind a residual sum that is still to be formed: the row is x + (acc + col_bias), written back on the way (`acc`
+// null: x + col_bias).
 template <typename TOut>
 __global__ void rmsnorm_pending_vec_kernel(float* x, const float* acc, const float* __restrict__ col_bias,
                                            const float* __restrict__ weight, float offset, TOut* __restrict__ out,
@@ -231,7 +232,7 @@ __global__ void rmsnorm_pending_vec_kernel(float* x, const float* acc, const flo
     }
     pdl_wait();
     float4* xr = reinterpret_cast<float4*>(after_wait(x) + (size_t)r * hidden);
-    const float4* ar = reinterpret_cast<const float4*>(after_wait(acc) + (size_t)r * hidden);
+    const float4* ar = acc ? reinterpret_cast<const float4*>(after_wait(acc) + (size_t)r * hidden) : nullptr;
     float4 kept[RMS_VEC];
     float s = 0.f;
 #pragma unroll
@@ -239,7 +240,7 @@ __global__ void rmsnorm_pending_vec_kernel(float* x, const float* acc, const flo
         const int i = threadIdx.x + n * blockDim.x;
         if (i < vecs) {
             const float4 a = xr[i];
-            float4 b = ar[i];
+            float4 b = ar ? ar[i] : make_float4(0.f, 0.f, 0.f, 0.f);
             if (col_bias) {
                 const float4 c = reinterpret_cast<const float4*>(col_bias)[i];
                 b.x += c.x; b.y += c.y; b.z += c.z; b.w += c.w;
@@ -327,6 +328,14 @@ __global__ void cast_rows_kernel(const float* __restrict__ x, __nv_bfloat16* __r
     if (i < count) out[i] = __float2bfloat16_rn(x[i]);
 }
 
+__global__ void add_row_kernel(float* x, const float* __restrict__ vector, int hidden) {
+    pdl_trigger();
+    const int i = blockIdx.y * blockDim.x + threadIdx.x;
+    const float v = i < hidden ? vector[i] : 0.f;
+    pdl_wait();
+    if (i < hidden) after_wait(x)[(size_t)blockIdx.x * hidden + i] += v;
+}
+
 __global__ void cast_columns_kernel(const float* __restrict__ x, int ld, __nv_bfloat16* __restrict__ out, int width,
                                     long long count) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -365,11 +374,18 @@ extern "C" int mx_rmsnorm(const float* x, const int* rows, const float* weight, 
 extern "C" int mx_epilogue(const void* acc, int acc_dtype, const float* bias, const float* residual, void* out,
                            int out_dtype, long long n_rows, int n_cols, int mode, cudaStream_t stream);
 
+// every row of x [n_rows][hidden] plus one vector
+extern "C" int mx_add_row(float* x, const float* vector, int n_rows, int hidden, cudaStream_t stream) {
+    if (n_rows <= 0 || hidden <= 0) return MX_OK;
+    mx_launch_chained(add_row_kernel, dim3(n_rows, (hidden + 255) / 256), dim3(256), 0, stream, x, vector, hidden);
+    return mx_launch_status();
+}
+
 extern "C" int mx_rmsnorm_pending(float* x, const float* acc, const float* col_bias, const float* weight, float offset,
                                   void* out, int out_dtype, int n_rows, int hidden, float eps, cudaStream_t stream) {
     if (n_rows <= 0) return MX_OK;
     if (hidden <= 0) MX_REFUSE("rmsnorm: hidden must be positive, got %d", hidden);
-    if (acc == nullptr) MX_REFUSE("rmsnorm of a pending sum: no accumulator");
+    if (acc == nullptr && col_bias == nullptr) MX_REFUSE("rmsnorm of a pending sum: nothing to add");
     const bool aligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(acc) |
                            reinterpret_cast<uintptr_t>(col_bias) | reinterpret_cast<uintptr_t>(weight) |
                            reinterpret_cast<uintptr_t>(out)) & 15) == 0;
@@ -384,7 +400,8 @@ extern "C" int mx_rmsnorm_pending(float* x, const float* acc, const float* col_b
         return mx_launch_status();
     }
     // rows that the float4 kernel does not take: the sum by the epilogue kernel, then the norm
-    const int rc = mx_epilogue(acc, MX_DTYPE_F32, col_bias, x, x, MX_DTYPE_F32, n_rows, hidden, MX_MODE_RESIDUAL, stream);
+    const int rc = acc ? mx_epilogue(acc, MX_DTYPE_F32, col_bias, x, x, MX_DTYPE_F32, n_rows, hidden, MX_MODE_RESIDUAL, stream)
+                       : mx_add_row(x, col_bias, n_rows, hidden, stream);
     if (rc != MX_OK) return rc;
     return mx_rmsnorm(x, nullptr, weight, offset, out, out_dtype, n_rows, hidden, eps, hidden, stream);
 }

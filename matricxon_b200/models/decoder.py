@@ -199,7 +199,7 @@ class DecoderModel:
             for position, entry in enumerate(schedule):
                 layer = self.layers[entry.layer]
                 if entry.pass_index is not None:
-                    if isinstance(x, PendingSum):
+                    if isinstance(x, PendingSum) and not self.pass_input.takes_pending_sum:
                         x = x.tensor()
                     x = self.pass_input.forward(x, entry.pass_index, ctx)
                 if isinstance(x, PendingSum) and not layer.takes_pending_sum:

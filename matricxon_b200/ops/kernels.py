@@ -570,15 +570,27 @@ def rmsnorm_sum(x: torch.Tensor, acc: torch.Tensor, alpha: float, weight: torch.
     _launched()
 
 
-def rmsnorm_pending(x: torch.Tensor, acc: torch.Tensor, col_bias: torch.Tensor | None, weight: torch.Tensor,
+def add_row(x: torch.Tensor, vector: torch.Tensor) -> None:
+    """``x += vector`` on every row, in place (float32)."""
+    _need(x, "x", torch.float32)
+    _need(vector, "vector", torch.float32)
+    assert vector.numel() == x.shape[1]
+    check(library().mx_add_row(_ptr(x), _ptr(vector), x.shape[0], x.shape[1], _stream()), "add_row")
+    _launched()
+
+
+def rmsnorm_pending(x: torch.Tensor, acc: torch.Tensor | None, col_bias: torch.Tensor | None, weight: torch.Tensor,
                     offset: float, eps: float, out: torch.Tensor) -> None:
-    """``x += acc + col_bias`` (the residual epilogue of a product whose float accumulator is ``acc``), then
+    """``x += acc + col_bias`` (the residual epilogue of a product whose float accumulator is ``acc``; None: the vector
+    alone), then
     ``out = x / sqrt(mean(x^2) + eps) * (offset + weight)``, in one pass over the rows."""
     _need(x, "x", torch.float32)
-    _need(acc, "acc", torch.float32)
+    if acc is not None:
+        _need(acc, "acc", torch.float32)
+        assert acc.shape == x.shape
     _need(weight, "weight", torch.float32)
     _need(out, "out")
-    assert acc.shape == x.shape and out.shape == x.shape and weight.numel() == x.shape[1]
+    assert out.shape == x.shape and weight.numel() == x.shape[1]
     if col_bias is not None:
         _need(col_bias, "col_bias", torch.float32)
         assert col_bias.numel() == x.shape[1]
@@ -1042,20 +1054,128 @@ def gla_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, decay: torc
 
 
 def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor,
-                  n_heads: int, vdim: int) -> None:
-    """out[t, h, e] = unit(o[t, h])[e] * weight[e] * silu(gate[t, h, e]); unit is the RMS norm over one head's
-    ``vdim`` entries with eps inside the root; ``weight`` None: no weight; ``gate`` a float32 view with any row stride."""
+                  n_heads: int, vdim: int, sigmoid_gate: bool = False, out_scale: float = 1.0,
+                  true_vdim: int | None = None) -> None:
+    """out[t, h, e] = out_scale * unit(o[t, h])[e] * weight[e] * silu(gate[t, h, e]); unit is the RMS norm over one head's
+    ``vdim`` entries (the mean divides by ``true_vdim`` where heads are filled up with zeros) with eps inside the root;
+    ``weight`` None: no weight; ``gate`` a float32 view with any row stride, as ``out``; ``sigmoid_gate``: sigmoid for silu."""
     _need(o, "o", torch.float32)
     _need(gate, "gate", torch.float32, contiguous=False)
     if weight is not None:
         _need(weight, "weight", torch.float32)
         assert weight.numel() == vdim
-    _need(out, "out")
+    _need(out, "out", contiguous=False)
     n = o.shape[0]
     assert tuple(o.shape) == (n, n_heads * vdim) and tuple(gate.shape) == (n, n_heads * vdim) and gate.stride(1) == 1
-    assert tuple(out.shape) == (n, n_heads * vdim)
+    assert tuple(out.shape) == (n, n_heads * vdim) and out.stride(1) == 1
     check(library().mx_gla_norm_gate(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), float(eps), _ptr(out),
-                                     dtype_code(out.dtype), n, n_heads, vdim, _stream()), "gla_norm_gate")
+                                     dtype_code(out.dtype), n, n_heads, vdim, 1 if sigmoid_gate else 0, out.stride(0),
+                                     float(out_scale), int(true_vdim or vdim), _stream()), "gla_norm_gate")
+    _launched()
+
+
+def norm_gate_rows(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor,
+                   sigmoid_gate: bool = False) -> None:
+    """out[t, e] = unit(o[t])[e] * weight[e] * silu(gate[t, e]) with one RMS norm over the whole row; ``gate`` and ``out``
+    may be strided; ``sigmoid_gate``: sigmoid for silu."""
+    _need(o, "o", torch.float32)
+    _need(gate, "gate", torch.float32, contiguous=False)
+    _need(out, "out", contiguous=False)
+    n, width = o.shape
+    assert gate.shape == o.shape == out.shape and gate.stride(1) == 1 == out.stride(1)
+    if weight is not None:
+        _need(weight, "weight", torch.float32)
+        assert weight.numel() == width
+    check(library().mx_norm_gate_rows(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), float(eps), _ptr(out),
+                                      dtype_code(out.dtype), n, width, 1 if sigmoid_gate else 0, out.stride(0), _stream()),
+          "norm_gate_rows")
+    _launched()
+
+
+# ---------------------------------------------------------------------- gated delta rule
+def delta_prepare(proj: torch.Tensor, b_col: int, a_col: int, conv: torch.Tensor, rate: torch.Tensor | None,
+                  dt_bias: torch.Tensor | None, state: torch.Tensor, tok_seq: torch.Tensor, cu_q: torch.Tensor,
+                  state_slots: torch.Tensor, qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor | None, qk_heads: int,
+                  heads: int, dim: int, vdim: int, q_scale: float, unit_eps: float) -> None:
+    """From float rows ``[q | k | v | ...]`` of a projection: a causal convolution per channel (``conv`` float32
+    [taps, channels], continuing from the start of ``state`` [slots, ...]), silu, q and k heads over their length (q times
+    ``q_scale``) into ``qkv`` [tokens, channels]; ``beta`` [tokens, heads] = sigmoid of the columns from ``b_col``; with
+    ``rate`` [heads] also ``decay`` [tokens, heads] = exp(rate * softplus(columns from a_col + dt_bias)). The state of
+    sequences that bring one token is moved on here, that of the others by ``conv_state_update`` afterwards."""
+    for name, tensor in (("proj", proj), ("conv", conv), ("state", state), ("qkv", qkv), ("beta", beta)):
+        _need(tensor, name, torch.float32, contiguous=name != "proj")
+    n, taps = proj.shape[0], conv.shape[0]
+    channels = 2 * qk_heads * dim + heads * vdim
+    assert proj.stride(1) == 1 and proj.shape[1] >= max(channels, b_col + heads, a_col + heads if rate is not None else 0)
+    assert conv.shape[1] == channels and tuple(qkv.shape) == (n, channels) and tuple(beta.shape) == (n, heads)
+    if rate is not None:
+        for name, tensor in (("rate", rate), ("dt_bias", dt_bias), ("decay", decay)):
+            _need(tensor, name, torch.float32)
+        assert rate.numel() == heads == dt_bias.numel() and tuple(decay.shape) == (n, heads)
+    check(library().mx_delta_prepare(
+        _ptr(proj), proj.stride(0), b_col, a_col, _ptr(conv), taps, _ptr(rate), _ptr(dt_bias) if rate is not None else None,
+        _ptr(state), state.stride(0), _ptr(tok_seq), _ptr(cu_q), _ptr(state_slots), _ptr(qkv), _ptr(beta),
+        _ptr(decay) if rate is not None else None, n, qk_heads, heads, dim, vdim, float(q_scale), float(unit_eps), _stream()),
+        "delta_prepare")
+    _launched()
+
+
+def delta_decay(low: torch.Tensor, a2: torch.Tensor, dt_bias: torch.Tensor, rate: torch.Tensor, decay: torch.Tensor) -> None:
+    """decay[t, h, d] = exp(rate[h] * softplus(a2[h, d] . low[t] + dt_bias[h, d])), all float32; ``low`` [tokens, rank] may
+    be a column range of wider rows; the rank is a multiple of four."""
+    _need(low, "low", torch.float32, contiguous=False)
+    for name, tensor in (("a2", a2), ("dt_bias", dt_bias), ("rate", rate), ("decay", decay)):
+        _need(tensor, name, torch.float32)
+    n, heads, dim = decay.shape
+    rank = low.shape[1]
+    assert low.shape[0] == n and low.stride(1) == 1 and a2.numel() == heads * dim * rank
+    assert dt_bias.numel() == heads * dim and rate.numel() == heads
+    check(library().mx_delta_decay(_ptr(low), low.stride(0), _ptr(a2), _ptr(dt_bias), _ptr(rate), _ptr(decay), n, heads * dim,
+                                   dim, rank, _stream()), "delta_decay")
+    _launched()
+
+
+def _delta_operands(qkv, beta, decay, state, state_offset, qk_heads, heads, dim, vdim):
+    for name, tensor in (("qkv", qkv), ("beta", beta), ("decay", decay), ("state", state)):
+        _need(tensor, name, torch.float32)
+    n = qkv.shape[0]
+    assert qkv.shape[1] == 2 * qk_heads * dim + heads * vdim and tuple(beta.shape) == (n, heads)
+    assert tuple(decay.shape) in ((n, heads), (n, heads, dim)) and state.stride(0) >= state_offset + heads * vdim * dim
+    return n, 1 if decay.dim() == 3 else 0
+
+
+def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, state_offset: int,
+               cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor, qk_heads: int, heads: int,
+               dim: int, vdim: int) -> None:
+    """``S <- g S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q`` over every sequence's tokens in order, from and to S
+    ([heads, vdim, dim] at ``state_offset`` of a sequence's ``state`` vector). ``decay`` [tokens, heads] or, one per key
+    channel, [tokens, heads, dim]; ``out`` float32 [tokens, heads * vdim]."""
+    n, per_channel = _delta_operands(qkv, beta, decay, state, state_offset, qk_heads, heads, dim, vdim)
+    _need(out, "out", torch.float32)
+    assert tuple(out.shape) == (n, heads * vdim)
+    check(library().mx_delta_scan(_ptr(qkv), _ptr(beta), _ptr(decay), per_channel, _ptr(state), state.stride(0),
+                                  int(state_offset), _ptr(cu_q), _ptr(state_slots), _ptr(out), n_seqs, qk_heads, heads, dim,
+                                  vdim, _stream()), "delta_scan")
+    _launched()
+
+
+def delta_step(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, state_offset: int,
+               cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, gate: torch.Tensor, sigmoid_gate: bool,
+               weight: torch.Tensor, eps: float, out: torch.Tensor, qk_heads: int, heads: int, dim: int, vdim: int,
+               out_scale: float = 1.0, true_vdim: int | None = None) -> None:
+    """``delta_scan`` and ``gla_norm_gate`` for steps in which no sequence brings more than one token; ``gate`` (float32)
+    and ``out`` (any activation dtype) [tokens, heads * vdim] may be strided."""
+    n, per_channel = _delta_operands(qkv, beta, decay, state, state_offset, qk_heads, heads, dim, vdim)
+    _need(gate, "gate", torch.float32, contiguous=False)
+    _need(weight, "weight", torch.float32)
+    _need(out, "out", contiguous=False)
+    assert tuple(gate.shape) == (n, heads * vdim) == tuple(out.shape) and gate.stride(1) == 1 == out.stride(1)
+    assert weight.numel() == vdim
+    check(library().mx_delta_step(_ptr(qkv), _ptr(beta), _ptr(decay), per_channel, _ptr(state), state.stride(0),
+                                  int(state_offset), _ptr(cu_q), _ptr(state_slots), _ptr(gate), gate.stride(0),
+                                  1 if sigmoid_gate else 0, _ptr(weight), float(eps), float(out_scale), _ptr(out),
+                                  dtype_code(out.dtype), out.stride(0), n_seqs, qk_heads, heads, dim, vdim,
+                                  int(true_vdim or vdim), _stream()), "delta_step")
     _launched()
 
 
@@ -1200,12 +1320,13 @@ def moe_combine(pairs: torch.Tensor, residual: torch.Tensor, top: int, identity=
 
 def moe_route_softmax(h: torch.Tensor, router: torch.Tensor, top: int, n_identity: int, correction: torch.Tensor | None,
                       ids: torch.Tensor, weights: torch.Tensor, counts: torch.Tensor, place: torch.Tensor,
-                      bias: torch.Tensor | None = None) -> None:
+                      bias: torch.Tensor | None = None, n_groups: int = 1, keep: int = 1) -> None:
     """Per token: softmax scores over the rows of the float32 router [experts + n_identity, K] (``bias``, float32 per
     row or None, is added to the logits first: with a bias and no correction the rule reads "the ``top`` largest
     logits, weighted by the softmax over those alone"); the ``top`` rows
     with the largest ``score + correction`` (float32 per row or None; ties to the lower index); weights = the
-    chosen rows' plain scores / their sum. ``counts`` [experts] must be zero; afterwards it holds every expert's
+    chosen rows' plain scores / their sum. With ``n_groups`` > 1 only rows of the ``keep`` runs of neighbours whose best
+    score is largest may be chosen. ``counts`` [experts] must be zero; afterwards it holds every expert's
     pairs and ``place`` each pair's index among them. A pair of one of the last ``n_identity`` rows keeps its id,
     is counted nowhere and has place 0."""
     _need(h, "h")
@@ -1224,7 +1345,7 @@ def moe_route_softmax(h: torch.Tensor, router: torch.Tensor, top: int, n_identit
         _need(bias, "bias", torch.float32)
         assert bias.numel() == router.shape[0]
     check(library().mx_moe_route_softmax(_ptr(h), dtype_code(h.dtype), h.stride(0), _ptr(router), k, n_experts, n_identity,
-                                         top, _ptr(correction), _ptr(bias), _ptr(ids), _ptr(weights), _ptr(counts), _ptr(place), n,
+                                         top, n_groups, keep, _ptr(correction), _ptr(bias), _ptr(ids), _ptr(weights), _ptr(counts), _ptr(place), n,
                                          _stream()), "moe_route_softmax")
     _launched()
 
@@ -1460,10 +1581,11 @@ def rotate_heads(rows: torch.Tensor, col: int, n_heads: int, dim: int, rot: int,
 def retention_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, head_decay: torch.Tensor, q_scale: float,
                    state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor,
                    n_heads: int, dim: int, vdim: int, positions: torch.Tensor | None = None,
-                   freq: torch.Tensor | None = None, rot: int = 0) -> None:
+                   freq: torch.Tensor | None = None, rot: int = 0, silu: bool = False) -> None:
     """``S <- head_decay_h S + k_t v_t^T; out_t = S^T (q_scale * q_t)`` over every sequence's tokens in order, from and
     to ``state`` [slots, heads, dim, vdim] (float32); q, k and v are column ranges of the float rows ``proj``. With
-    ``freq`` q and k are rotated over their first ``rot`` entries on their way in."""
+    ``freq`` q and k are rotated over their first ``rot`` entries on their way in; with ``silu`` q, k and v are the silu of
+    what the rows hold (unrotated heads)."""
     for name, tensor in (("proj", proj), ("head_decay", head_decay), ("state", state), ("out", out)):
         _need(tensor, name, torch.float32)
     n = proj.shape[0]
@@ -1475,8 +1597,8 @@ def retention_scan(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, head_
         assert freq.numel() >= rot // 2 and positions.numel() >= n
     check(library().mx_retention_scan(_ptr(proj), proj.stride(0), q_col, k_col, v_col, _ptr(head_decay), float(q_scale),
                                       _ptr(state), _ptr(cu_q), _ptr(state_slots), _ptr(out), n_seqs, n_heads, dim, vdim,
-                                      _ptr(positions) if freq is not None else None, _ptr(freq), int(rot), _stream()),
-          "retention_scan")
+                                      _ptr(positions) if freq is not None else None, _ptr(freq), int(rot), 1 if silu else 0,
+                                      _stream()), "retention_scan")
     _launched()
 
 
@@ -1488,16 +1610,17 @@ def retention_chunked(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_
                       q_scale: float, eps: float, state: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor,
                       n_seqs: int, chunks: torch.Tensor, seq_chunk0: torch.Tensor, n_chunks: int, out: torch.Tensor,
                       n_heads: int, dim: int, vdim: int, positions: torch.Tensor | None = None,
-                      freq: torch.Tensor | None = None, rot: int = 0) -> None:
+                      freq: torch.Tensor | None = None, rot: int = 0, silu: bool = False, raw: bool = False) -> None:
     """``retention_scan`` and ``gla_norm_gate`` (without a weight) for long portions, in chunks of
     ``retention_chunk_tokens()`` tokens (``scan_chunk_lists`` on the device) whose products run in parallel on the FP32
     cores: ``out`` [tokens, heads * vdim] (any activation dtype, rows may be strided) = unit(o) * silu(gate), ``gate`` being
-    the columns from ``g_col`` of the float rows ``proj``. Heads of at most 128 x 128."""
+    the columns from ``g_col`` of the float rows ``proj``. ``silu`` as in ``retention_scan``; ``raw``: ``out`` is o itself,
+    float32, without norm and gate. Heads of at most 128 x 128."""
     for name, tensor in (("proj", proj), ("head_decay", head_decay), ("state", state)):
         _need(tensor, name, torch.float32, contiguous=name != "proj")
     for name, tensor in (("chunks", chunks), ("seq_chunk0", seq_chunk0), ("cu_q", cu_q), ("state_slots", state_slots)):
         _need(tensor, name, torch.int32)
-    _need(out, "out", contiguous=False)
+    _need(out, "out", torch.float32 if raw else None, contiguous=False)
     n = proj.shape[0]
     assert tuple(state.shape[1:]) == (n_heads, dim, vdim), state.shape
     assert proj.stride(1) == 1 and proj.shape[1] >= g_col + n_heads * vdim and head_decay.numel() == n_heads
@@ -1514,8 +1637,8 @@ def retention_chunked(proj: torch.Tensor, q_col: int, k_col: int, v_col: int, g_
                                          float(q_scale), float(eps), _ptr(positions) if freq is not None else None,
                                          _ptr(freq), int(rot), _ptr(state), _ptr(cu_q), _ptr(state_slots), n_seqs,
                                          _ptr(chunks), _ptr(seq_chunk0), n_chunks, _ptr(scratch), _ptr(out),
-                                         dtype_code(out.dtype), out.stride(0), n_heads, dim, vdim, _stream()),
-          "retention_chunked")
+                                         dtype_code(out.dtype), out.stride(0), n_heads, dim, vdim, 1 if silu else 0,
+                                         1 if raw else 0, _stream()), "retention_chunked")
     _launched(3)
 
 

@@ -46,6 +46,7 @@ _SIGNATURES: dict[str, tuple[list, object]] = {
     "mx_paged_attention_tc_split": ([P, I, P, L, I, P, I, P, P, P, I, I, I, I, I, I, F, P, I, I, P, P, F, P, I, P, P], I),
     "mx_paged_attention": ([P, I, I, P, L, I, P, I, P, P, I, I, I, I, I, F, P, I, I, P, P, F, P, I, P, P], I),
     "mx_rmsnorm": ([P, P, P, F, P, I, I, I, F, L, P], I),
+    "mx_add_row": ([P, P, I, I, P], I),
     "mx_rmsnorm_pending": ([P, P, P, P, F, P, I, I, I, F, P], I),
     "mx_rmsnorm_branch_add": ([P, P, P, P, P, I, I, I, F, P], I),
     "mx_rmsnorm_sum": ([P, P, F, P, F, P, I, I, I, F, P], I),
@@ -66,9 +67,9 @@ _SIGNATURES: dict[str, tuple[list, object]] = {
     "mx_head_gate": ([P, P, I, P, I, I, I, I, I, P], I),
     "mx_gla_decay": ([P, I, P, P, F, P, I, I, I, P], I),
     "mx_gla_scan": ([P, I, I, I, I, P, F, P, P, P, P, I, I, I, I, P], I),
-    "mx_retention_scan": ([P, I, I, I, I, P, F, P, P, P, P, I, I, I, I, P, P, I, P], I),
+    "mx_retention_scan": ([P, I, I, I, I, P, F, P, P, P, P, I, I, I, I, P, P, I, I, P], I),
     "mx_retention_chunk_tokens": ([], I),
-    "mx_retention_chunked": ([P, I, I, I, I, I, P, F, F, P, P, I, P, P, P, I, P, P, I, P, P, I, I, I, I, I, P], I),
+    "mx_retention_chunked": ([P, I, I, I, I, I, P, F, F, P, P, I, P, P, P, I, P, P, I, P, P, I, I, I, I, I, I, I, P], I),
     "mx_rotate_heads": ([P, I, I, I, I, I, I, P, P, P], I),
     "mx_conv_norm_kv_write": ([P, I, P, P, I, P, P, F, F, F, P, L, P, P, P, P, P, P, L, I, P, I, I, I, I, I, I, I, I, P, P], I),
     "mx_conv_state_update": ([P, I, I, P, P, L, P, P, I, I, I, P], I),
@@ -76,9 +77,14 @@ _SIGNATURES: dict[str, tuple[list, object]] = {
     "mx_selective_scan": ([P, P, I, P, I, P, P, P, P, I, I, P, L, L, P, P, P, I, I, I, I, I, I, F, P], I),
     "mx_selective_scan_chunked": ([P, P, I, P, I, P, P, P, P, I, I, P, L, L, P, P, P, I, I, I, I, I, I, F, P, P, I, I, P, P], I),
     "mx_selective_step": ([P, P, I, P, P, P, P, P, I, I, P, L, L, P, P, P, I, I, I, I, I, I, F, P], I),
-    "mx_gla_norm_gate": ([P, P, I, P, F, P, I, I, I, I, P], I),
+    "mx_gla_norm_gate": ([P, P, I, P, F, P, I, I, I, I, I, I, F, I, P], I),
+    "mx_norm_gate_rows": ([P, P, I, P, F, P, I, I, I, I, I, P], I),
+    "mx_delta_prepare": ([P, I, I, I, P, I, P, P, P, L, P, P, P, P, P, P, I, I, I, I, I, F, F, P], I),
+    "mx_delta_decay": ([P, I, P, P, P, P, I, I, I, I, P], I),
+    "mx_delta_scan": ([P, P, P, I, P, L, L, P, P, P, I, I, I, I, I, P], I),
+    "mx_delta_step": ([P, P, P, I, P, L, L, P, P, P, I, I, P, F, F, P, I, I, I, I, I, I, I, I, P], I),
     "mx_moe_route": ([P, I, I, P, I, I, I, I, I, F, I, P, P, P, P, I, P], I),
-    "mx_moe_route_softmax": ([P, I, I, P, I, I, I, I, P, P, P, P, P, P, I, P], I),
+    "mx_moe_route_softmax": ([P, I, I, P, I, I, I, I, I, I, P, P, P, P, P, P, I, P], I),
     "mx_moe_tile_rows": ([], I),
     "mx_moe_plan": ([P, P, P, I, I, I, P, P, P, P, P], I),
     "mx_moe_gather": ([P, I, P, I, P, I, I, P], I),

@@ -89,9 +89,9 @@ class PendingSum:
     """``residual + x @ W.T + bias`` not yet added up: the library's float product of a step with 17 or
     more rows, handed to the norm that follows, which forms the sum on its way through the rows
     (``kernels.layernorm_sum``) instead of an epilogue pass of its own. ``tensor()`` adds it up for
-    anybody else."""
+    anybody else. ``acc`` None: only a vector (``bias``) is still to be added to every row."""
 
-    def __init__(self, acc: torch.Tensor, bias: torch.Tensor | None, residual: torch.Tensor) -> None:
+    def __init__(self, acc: torch.Tensor | None, bias: torch.Tensor | None, residual: torch.Tensor) -> None:
         self.acc, self.bias, self.residual = acc, bias, residual
         self._done = False
 
@@ -113,7 +113,9 @@ class PendingSum:
         return self.residual
 
     def tensor(self) -> torch.Tensor:
-        if not self._done:
+        if not self._done and self.acc is None:
+            kernels.add_row(self.residual, self.bias)
+        elif not self._done:
             kernels.epilogue(self.acc, self.bias, self.residual, self.residual, EPILOGUE_RESIDUAL)
             self._done = True
         return self.residual

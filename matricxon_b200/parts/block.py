@@ -9,6 +9,8 @@ and each sub-layer adds into it in float.
 ``branch_norm_sequential``: ``x = x + s1 * norm1(mixer(x)); x = x + s2 * norm2(ffn(x))`` with learned vectors
 ``s1``, ``s2`` (optional), then whatever the layer adds from outside the stream (``LayerSpec.side_input``).
 
+``pre_norm_parallel``: ``h = norm(x); x = x + mixer(h) + ffn(h)``: one norm, read by both sublayers.
+
 ``sandwich_norm_sequential``: ``x = x + norm1b(mixer(norm1(x))); x = x + norm2b(ffn(norm2(x)))``: a norm before and
 one after each sublayer.
 """
@@ -80,6 +82,58 @@ class PreNormSequentialBlock(Block):
             if self.feed_forward is not None:
                 x, h = self._normed(self.ffn_norm, x)
                 x = self.feed_forward.forward(h, x, ctx)
+        finally:
+            ctx.sums_may_pend = False
+        if isinstance(x, PendingSum) and not getattr(ctx, "pending_sum_wanted", False):
+            return x.tensor()
+        return x
+
+
+@register_part("block", "pre_norm_parallel")
+class PreNormParallelBlock(Block):
+    """``h = norm(x); x = x + (mixer(h) + ffn(h))``: mixer and feed-forward read the same rows. Both add into the float
+    stream, the feed-forward first: what the mixer's output product leaves pending the next norm adds up. A layer may
+    have no feed-forward."""
+
+    takes_pending_sum = True
+
+    def __init__(self, spec, runtime, prefix):
+        super().__init__(spec, runtime, prefix)
+        sep = spec.part_separator
+        self.mixer_norm = build_part("norm", spec.mixer_norm, runtime, f"{prefix}{spec.mixer_norm_name}{sep}")
+        self.mixer = build_part("mixer", spec.mixer, runtime, f"{prefix}{spec.mixer_name}{sep}")
+        self.feed_forward = None
+        if spec.feed_forward is not None:
+            self.feed_forward = build_part("feed_forward", spec.feed_forward, runtime,
+                                           f"{prefix}{spec.feed_forward_name}{sep}")
+        self.capturable = all(part.capturable for part in self.parts())
+
+    @classmethod
+    def weight_specs(cls, spec, prefix):
+        from matricxon_b200.parts.base import part_class
+
+        groups = [("norm", spec.mixer_norm, spec.mixer_norm_name), ("mixer", spec.mixer, spec.mixer_name)]
+        if spec.feed_forward is not None:
+            groups.append(("feed_forward", spec.feed_forward, spec.feed_forward_name))
+        out = []
+        for category, sub, name in groups:
+            out.extend(part_class(category, sub.kind).weight_specs(sub, f"{prefix}{name}{spec.part_separator}"))
+        return out
+
+    def parts(self):
+        return tuple(part for part in (self.mixer_norm, self.mixer, self.feed_forward) if part is not None)
+
+    def load(self, fetch):
+        for part in self.parts():
+            part.load(fetch)
+
+    def forward(self, x, ctx, binding):
+        x, h = PreNormSequentialBlock._normed(self.mixer_norm, x)
+        if self.feed_forward is not None:
+            x = self.feed_forward.forward(h, x, ctx)
+        ctx.sums_may_pend = True
+        try:
+            x = self.mixer.forward(h, x, ctx, binding)
         finally:
             ctx.sums_may_pend = False
         if isinstance(x, PendingSum) and not getattr(ctx, "pending_sum_wanted", False):

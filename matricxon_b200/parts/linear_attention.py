@@ -14,7 +14,8 @@ and the gate are float in both dtypes; only the large projections run in the run
 Retention (``RetentionSpec``) decays by one constant per head: ``S_t = decay_h S_(t-1) + k_t v_t^T``, ``o_t = S_t^T q_t`` with
 q and k rotated over their first entries. It shares the recurrence's kernel (which takes no decay operand then), the
 state's layout and the kernel behind it (no weight in its norm); short portions are rotated by a pass of their own, steps
-of one token a sequence on the operands' way into the recurrence. Long portions of heads of up to 128 x 128 run in chunks
+of one token a sequence on the operands' way into the recurrence. In another form (lightning attention) q, k and v are the
+silu of their projections, taken on the operands' way in, and one norm with a weight spans all heads. Long portions of heads of up to 128 x 128 run in chunks
 of tokens whose products take the place of the updates, with rotation, norm and gate in the same kernels.
 """
 
@@ -98,6 +99,9 @@ class Retention(BranchMixer):
                                           or getattr(self.position, "interleaved", False)
                                           or getattr(self.position, "amplitude", 1.0) != 1.0):
             raise ValueError(f"retention rotates by a plain table with halves paired, not by {spec.position!r}")
+        if self.position is not None and spec.activation is not None:
+            raise ValueError("activated heads are not rotated by any kernel")
+        self.silu, self.sigmoid_gate, self.joint = spec.activation == "silu", spec.gate == "sigmoid", spec.norm == "all"
 
     @classmethod
     def _matrices(cls, spec):
@@ -108,6 +112,9 @@ class Retention(BranchMixer):
     def weight_specs(cls, spec, prefix):
         specs = [WeightSpec(prefix + name, (rows, spec.hidden_size), role="matrix", init="weight")
                  for name, rows in cls._matrices(spec)]
+        if spec.norm_name is not None:
+            specs.append(WeightSpec(prefix + spec.norm_name, (spec.num_heads * spec.value_dim,), role="vector",
+                                    init="norm_weight"))
         specs.append(WeightSpec(prefix + spec.output_name, (spec.hidden_size, spec.num_heads * spec.value_dim),
                                 role="matrix", init="weight"))
         return specs
@@ -120,6 +127,7 @@ class Retention(BranchMixer):
         p, s = self.prefix, self.spec
         self.input_weight = torch.cat([fetch(p + name) for name, _ in self._matrices(s)])
         self.output_weight = fetch(p + s.output_name)
+        self.norm_weight = fetch(p + s.norm_name) if s.norm_name is not None else None
         self.decay = torch.tensor(s.decay, dtype=torch.float32, device=self.runtime.device)
 
     def mix(self, proj, ctx, binding, out, scale=1.0):
@@ -143,9 +151,14 @@ class Retention(BranchMixer):
                 ctx.memo[key] = (both[:len(chunks)], both[len(chunks):], len(chunks) // 2)
             if self.position is not None:
                 rotation = {"positions": ctx.positions, "freq": freq, "rot": rot}
+            # the kernel ends in a silu-gated norm of every head; another ending follows it as a kernel of its own
+            raw = self.joint or self.sigmoid_gate
+            o = torch.empty((n, values), dtype=torch.float32, device=proj.device) if raw else out
             kernels.retention_chunked(proj, 0, keys, 2 * keys, 2 * keys + values, self.decay, s.key_scale, s.eps,
-                                      binding.state, ctx.cu_q, ctx.state_slots, ctx.n_seqs, *ctx.memo[key], out,
-                                      s.num_heads, s.head_dim, s.value_dim, **rotation)
+                                      binding.state, ctx.cu_q, ctx.state_slots, ctx.n_seqs, *ctx.memo[key], o,
+                                      s.num_heads, s.head_dim, s.value_dim, silu=self.silu, raw=raw, **rotation)
+            if raw:
+                self._norm_gate(o, proj, out)
             return
         if self.position is not None:
             if one_token_each(ctx):
@@ -155,9 +168,14 @@ class Retention(BranchMixer):
         o = torch.empty((n, values), dtype=torch.float32, device=proj.device)
         # the scale of k goes on q: the output is linear in both, and the state then holds the plain k v^T
         kernels.retention_scan(proj, 0, keys, 2 * keys, self.decay, s.key_scale, binding.state, ctx.cu_q, ctx.state_slots,
-                               ctx.n_seqs, o, s.num_heads, s.head_dim, s.value_dim, **rotation)
+                               ctx.n_seqs, o, s.num_heads, s.head_dim, s.value_dim, silu=self.silu, **rotation)
+        self._norm_gate(o, proj, out)
+
+    def _norm_gate(self, o, proj, out):
+        s = self.spec
+        keys, values = s.num_heads * s.head_dim, s.num_heads * s.value_dim
         gate = proj[:, 2 * keys + values:2 * keys + 2 * values]
-        rows = out if out.is_contiguous() else torch.empty(tuple(out.shape), dtype=out.dtype, device=out.device)
-        kernels.gla_norm_gate(o, gate, None, s.eps, rows, s.num_heads, s.value_dim)
-        if rows is not out:
-            out.copy_(rows)
+        if self.joint:
+            kernels.norm_gate_rows(o, gate, self.norm_weight, s.eps, out, sigmoid_gate=self.sigmoid_gate)
+        else:
+            kernels.gla_norm_gate(o, gate, None, s.eps, out, s.num_heads, s.value_dim, sigmoid_gate=self.sigmoid_gate)

@@ -51,6 +51,11 @@ class ParallelMixer(Mixer):
         for branch, _ in self.branches:
             branch.load(fetch)
         parts = [branch for branch, _ in self.branches]
+        for branch in parts:
+            # every branch's columns of the input product start on a 16-byte boundary
+            short = -branch.input_weight.shape[0] % 8
+            if short:
+                branch.input_weight = torch.nn.functional.pad(branch.input_weight, (0, 0, 0, short))
         self.input_rows = [branch.input_weight.shape[0] for branch in parts]
         self.output_columns = [branch.output_weight.shape[1] for branch in parts]
         self.input_weight = torch.cat([branch.input_weight for branch in parts])

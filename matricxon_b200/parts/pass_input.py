@@ -1,5 +1,8 @@
 """What a model does to the stream before every pass of a repeated run of layers.
 
+``StepVectorSpec``: ``x <- x + s_t``. The sum is left to the norm that reads the stream next (``ops.linear.PendingSum``),
+beside whatever sum the layer before left pending there.
+
 ``ReinjectionSpec``: with x0 the embedding output of the step's tokens and t the number of the pass,
 ``x <- M [x; x0] + s_t``. M is split by columns at load, ``M = [A | B]``: ``B x0`` is the same for every pass and is
 formed once per step, right after the embedding lookup (``begin``), so the stream's buffer may be overwritten by the
@@ -12,7 +15,7 @@ from __future__ import annotations
 import torch
 
 from matricxon_b200.ops import kernels
-from matricxon_b200.ops.linear import EPILOGUE_F32, EPILOGUE_RESIDUAL, linear
+from matricxon_b200.ops.linear import EPILOGUE_F32, EPILOGUE_RESIDUAL, PendingSum, linear
 from matricxon_b200.parts.base import Part, register_part
 from matricxon_b200.weights.loader import WeightSpec
 
@@ -20,6 +23,9 @@ from matricxon_b200.weights.loader import WeightSpec
 class PassInput(Part):
     """``begin(x0, ctx)`` sees the embedding output before any layer runs; ``forward(x, pass_index, ctx) -> x`` runs
     before the schedule entry that opens a pass (the result may be a new buffer)."""
+
+    # True: ``forward`` takes an ``ops.linear.PendingSum`` for the stream, and may return one
+    takes_pending_sum = False
 
     def begin(self, x0, ctx):
         return None
@@ -70,3 +76,26 @@ class Reinjection(PassInput):
         out = torch.empty_like(base)
         return linear(self._activations(x, ctx), self.stream_weight, self.steps[pass_index], EPILOGUE_RESIDUAL,
                       residual=base, out=out, backend=self.runtime.gemm_backend)
+
+
+@register_part("pass_input", "step_vector")
+class StepVector(PassInput):
+    capturable = True
+    takes_pending_sum = True
+
+    @classmethod
+    def weight_specs(cls, spec, prefix):
+        return [WeightSpec(prefix + spec.step_name, (spec.passes, spec.hidden_size), role="vector", init="bias")]
+
+    def load(self, fetch):
+        self.steps = fetch(self.prefix + self.spec.step_name)
+
+    def forward(self, x, pass_index, ctx):
+        if not 0 <= pass_index < self.spec.passes:
+            raise ValueError(f"pass {pass_index} of a run of {self.spec.passes}")
+        step = self.steps[pass_index]
+        if isinstance(x, PendingSum):
+            if x.bias is None:
+                return PendingSum(x.acc, step, x.residual)
+            x = x.tensor()
+        return PendingSum(None, step, x)

@@ -15,7 +15,7 @@ second weighs every pair's row). The experts' matrices are stacked at load: ``[e
 
 ``score="softmax"`` routes by another rule (softmax over all router rows, a correction that moves the choice and not
 the weights; optionally a bias on the logits themselves, which makes the rule "the largest logits, weighted by the
-softmax over the chosen ones") and may name experts without matrices that return their input: such a pair takes no row of the grouped
+softmax over the chosen ones"; optionally limited to the groups of neighbours whose best score is largest) and may name experts without matrices that return their input: such a pair takes no row of the grouped
 products, and the combining kernel adds ``weight * h`` for it. An expert may be a ``GatedMlpSpec`` or a
 ``ClampedGluSpec`` (the activation differs). ``weight_on="input"`` puts a pair's weight on the expert's input instead of
 its output, ``normalize=False`` leaves the sigmoid scores as the weights. A ``shared`` feed-forward runs for every token; the routed sum is added
@@ -102,7 +102,7 @@ class RoutedExperts(FeedForward):
         weights = torch.empty(n_pairs, dtype=torch.float32, device=device)
         if s.score == "softmax":
             kernels.moe_route_softmax(h, self.router, s.top, s.num_identity, self.correction, ids, weights, counts, place,
-                                      bias=self.bias)
+                                      bias=self.bias, n_groups=s.num_groups, keep=s.groups_kept)
         else:
             kernels.moe_route(h, self.router, s.top, s.num_groups, s.groups_kept, s.route_scale, ids, weights, counts,
                               place, normalize=s.normalize)

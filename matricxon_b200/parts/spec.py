@@ -576,7 +576,11 @@ class RetentionSpec:
     """Linear attention with a constant decay per head: q and k (``head_dim`` wide) rotated over their first entries
     (``position``; None: not), ``k`` times ``key_scale``; ``S <- decay_h S + k_t v_t^T`` from S = 0, ``o_t = S^T q_t``;
     every head's o is divided by its root mean square over ``value_dim`` (eps inside, no weight), the heads are
-    multiplied by ``silu(W_g h)`` and projected by W_o. No biases."""
+    multiplied by ``silu(W_g h)`` and projected by W_o. No biases.
+
+    ``activation="silu"``: q, k and v are the silu of their projections. ``norm="all"``: the concatenated heads are divided
+    by one root mean square over all of them, times a plain weight (``norm_name``, heads * value_dim entries; it may be
+    None). ``gate``: ``"silu"`` or ``"sigmoid"``."""
 
     hidden_size: int
     num_heads: int
@@ -591,17 +595,86 @@ class RetentionSpec:
     value_name: str
     gate_name: str
     output_name: str
+    activation: str | None = None
+    norm: str = "head"
+    norm_name: str | None = None
+    gate: str = "silu"
     kind: str = "retention"
 
     def __post_init__(self) -> None:
         if min(self.num_heads, self.head_dim, self.value_dim) <= 0:
             raise ValueError("retention needs positive head count and head sizes")
+        if self.activation not in (None, "silu") or self.norm not in ("head", "all") or self.gate not in ("silu", "sigmoid"):
+            raise ValueError("retention: activation None or 'silu', norm 'head' or 'all', gate 'silu' or 'sigmoid'")
+        if self.norm_name is not None and self.norm != "all":
+            raise ValueError("a retention norm with a weight spans all heads")
         if self.head_dim > 256:
             raise ValueError(f"{self.head_dim} key channels per head: the recurrence kernel takes up to 256")
         if len(self.decay) != self.num_heads:
             raise ValueError(f"{len(self.decay)} decays for {self.num_heads} heads")
         if self.position is not None and self.position.rotary_dim > self.head_dim:
             raise ValueError(f"{self.position.rotary_dim} rotated entries exceed the head of {self.head_dim}")
+
+
+@dataclass(frozen=True)
+class DeltaRuleSpec:
+    """Linear attention by the gated delta rule. q and k (``num_kv_heads`` heads of ``head_dim``) and v (``num_heads`` heads
+    of ``value_dim``) are projections that pass a causal convolution over time per channel (``taps``, the last on the
+    current token, no bias) and silu; q and k are then divided by their length, ``x / sqrt(sum x^2 + unit_eps)``, and q
+    is multiplied by ``query_scale``; value head h reads q/k head ``h // (num_heads / num_kv_heads)``. Per value head
+    ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q`` from S = 0 with ``beta = sigmoid(W_b h)`` and a
+    decay ``g = exp(-exp(A_log_h) softplus(z + dt_bias))``:
+
+    ``decay="head"``: one g per head, ``z = W_a h`` (``decay_names`` = (W_a,)); ``decay="channel"``: one per head and key
+    channel (a row of S), ``z = A2 (A1 h)`` (``decay_names`` = (A1, A2), ``decay_rank`` between them).
+
+    Every head's o is divided by its root mean square over ``value_dim`` (``eps`` inside) times one weight shared by the
+    heads, times ``act(gate)`` with ``gate`` one of ``"silu"`` / ``"sigmoid"``, its logits ``W_g h`` (``gate_names`` =
+    (W_g,)) or ``G2 (G1 h)`` (``gate_names`` = (G1, G2), ``gate_rank`` between them); then W_o. Names are full tensor names
+    under the mixer's prefix; a convolution is its projection's name with ``conv_suffix``."""
+
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    taps: int
+    eps: float
+    query_scale: float
+    decay: str
+    gate: str
+    query_name: str
+    key_name: str
+    value_name: str
+    beta_name: str
+    a_log_name: str
+    dt_bias_name: str
+    decay_names: tuple[str, ...]
+    gate_names: tuple[str, ...]
+    norm_name: str
+    output_name: str
+    decay_rank: int | None = None
+    gate_rank: int | None = None
+    unit_eps: float = 1e-6
+    conv_suffix: str = ".conv"
+    kind: str = "delta_rule"
+
+    def __post_init__(self) -> None:
+        if min(self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim) <= 0 or self.num_heads % self.num_kv_heads:
+            raise ValueError(f"the delta rule needs positive head sizes and value heads ({self.num_heads}) in a multiple of "
+                             f"the q/k heads ({self.num_kv_heads})")
+        if self.head_dim > 256:
+            raise ValueError(f"{self.head_dim} key channels per head: the recurrence kernel takes up to 256")
+        if not 1 <= self.taps <= 16:
+            raise ValueError(f"a convolution of {self.taps} taps: the kernel takes 1 to 16")
+        if self.decay not in ("head", "channel") or self.gate not in ("silu", "sigmoid"):
+            raise ValueError("decay is 'head' or 'channel', gate 'silu' or 'sigmoid'")
+        if len(self.decay_names) != (1 if self.decay == "head" else 2):
+            raise ValueError("a decay per head has one matrix, a decay per channel two")
+        if len(self.decay_names) == 2 and not 0 < (self.decay_rank or 0) <= 768:
+            raise ValueError(f"a decay rank of {self.decay_rank}: the decay kernel takes 1 to 768")
+        if len(self.gate_names) not in (1, 2) or (len(self.gate_names) == 2 and not (self.gate_rank or 0) > 0):
+            raise ValueError("a gate has one matrix, or two and the rank between them")
 
 
 @dataclass(frozen=True)
@@ -630,6 +703,21 @@ class ReinjectionSpec:
     matrix_name: str
     step_name: str
     kind: str = "reinjection"
+
+    def __post_init__(self) -> None:
+        if self.passes <= 0:
+            raise ValueError(f"a repeated run has at least one pass, got {self.passes}")
+
+
+@dataclass(frozen=True)
+class StepVectorSpec:
+    """What a model adds to the stream before every pass of a repeated run of layers: row t of ``step_name``
+    ([passes, hidden], a full tensor name) before pass t."""
+
+    hidden_size: int
+    passes: int
+    step_name: str
+    kind: str = "step_vector"
 
     def __post_init__(self) -> None:
         if self.passes <= 0:
@@ -696,7 +784,8 @@ class RoutedExpertsSpec:
 
     ``score="softmax"`` is another rule: scores are the softmax over all router rows, the ``top`` rows with the
     largest ``score + correction`` win (``correction_name``: a float per row, None: none) and the weights use the
-    plain scores; there are no groups and no ``route_scale``. The router then has ``num_experts + num_identity``
+    plain scores; there is no ``route_scale``. Groups are ranked by their ``group_best`` = 1 largest score there, and go
+    with routers that have neither a correction nor experts without tensors. The router then has ``num_experts + num_identity``
     rows, the last ``num_identity`` of which stand for experts without tensors whose output is their input.
     ``expert`` may be a ``GatedMlpSpec`` or a ``ClampedGluSpec``. ``shared`` (a feed-forward spec, tensors under
     ``<prefix><shared_name>``) runs for every token and is added. With ``bias_name`` the logits are ``R h + b``; the
@@ -744,13 +833,17 @@ class RoutedExpertsSpec:
                                         or self.bias_name is not None):
             raise ValueError("experts without tensors, a correction of the choice and a bias on the logits belong "
                              "to the softmax rule")
-        if self.score == "softmax" and (self.num_groups != 1 or self.route_scale != 1.0):
-            raise ValueError("the softmax rule has neither groups nor a scale of its weights")
+        if self.score == "softmax" and self.route_scale != 1.0:
+            raise ValueError("the softmax rule has no scale of its weights")
+        if self.score == "softmax" and self.num_groups != 1 and (
+                self.group_best != 1 or self.num_identity or self.correction_name is not None or self.bias_name is not None):
+            raise ValueError("the softmax rule ranks groups by their best score, without corrections and experts that have "
+                             "no tensors")
         if not 0 < self.top <= self.num_experts + self.num_identity:
             raise ValueError(f"a token cannot run {self.top} of {self.num_experts + self.num_identity} experts")
-        if self.score == "softmax":
-            if self.norm_eps != 1e-20:
-                raise ValueError("the routing kernel adds 1e-20 to the sum")
+        if self.norm_eps != 1e-20:
+            raise ValueError("the routing kernel adds 1e-20 to the sum")
+        if self.score == "softmax" and self.num_groups == 1:
             return
         if self.num_groups <= 0 or self.num_experts % self.num_groups:
             raise ValueError(f"{self.num_experts} experts cannot form {self.num_groups} equal groups")
@@ -758,8 +851,8 @@ class RoutedExpertsSpec:
             raise ValueError(f"{self.groups_kept} of {self.num_groups} groups cannot be kept")
         if self.groups_kept * (self.num_experts // self.num_groups) < self.top:
             raise ValueError(f"{self.groups_kept} kept groups hold fewer than {self.top} experts")
-        if self.group_best != 2 or self.norm_eps != 1e-20:
-            raise ValueError("the routing kernel ranks groups by their two best scores and adds 1e-20 to the sum")
+        if self.score == "sigmoid" and self.group_best != 2:
+            raise ValueError("the sigmoid rule ranks groups by their two best scores")
 
 
 @dataclass(frozen=True)
@@ -791,7 +884,7 @@ class LayerSpec:
     ffn_out_norm: Any | None = None
     mixer_out_norm_name: str = ""
     ffn_out_norm_name: str = ""
-    # what the pre-norm block puts behind a part's name fragment to make its prefix ("" for checkpoints whose
+    # what the pre-norm blocks puts behind a part's name fragment to make its prefix ("" for checkpoints whose
     # fragments carry their own separators, as the post-norm block expects them)
     part_separator: str = "."
 
@@ -835,7 +928,8 @@ class ModelSpec:
     head_bias: bool = False
     logit_softcap: float | None = None
     logit_scale: float = 1.0             # logits times a constant
-    # what happens to the stream before the schedule entries that open a pass (``ReinjectionSpec``; None: nothing)
+    # what happens to the stream before the schedule entries that open a pass (``ReinjectionSpec`` or
+    # ``StepVectorSpec``; None: nothing)
     pass_input: Any | None = None
     # how names are put together: "<embedding_name><weight_suffix>", a layer's prefix from
     # ``layer_prefix_format`` (fields {prefix} and {index}), the final norm's prefix (None:
