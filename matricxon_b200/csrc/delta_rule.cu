@@ -17,10 +17,14 @@
 //   that bring one token is moved on here, that of the others by mx_conv_state_update afterwards.
 // mx_delta_decay: g for every head and key channel from a low-rank row: exp(rate_h softplus(A2 low + dt_bias)); a thread per
 //   channel keeps its row of A2 in registers for sixteen tokens.
-// mx_delta_scan: every sequence's tokens in order. A block owns (sequence, head, 16 value columns); eight lanes share a
-//   column, each with an eighth of its rows in registers for the whole portion. Tokens arrive in rounds by cp.async, two
-//   rounds in flight; S^T k is reduced by three shuffles a token, the shares of the read-outs meet in shared memory once a
-//   round.
+// mx_delta_scan: every sequence's tokens in order, eight at a time. Within a group of eight the writes u solve a triangular
+//   system whose coefficients do not depend on the state: u = T (v - S^T k'), o = S^T q' + P u, S <- G S + k'' u^T with k', q'
+//   decayed from the group's start, k'' to its end, G over the whole group, T and P 8 x 8. A first kernel forms them for
+//   all groups in parallel (decays enter as products of numbers up to one, nothing is divided); the second walks the
+//   groups: a block owns (sequence, head, 16 value columns), sixteen lanes share two columns with their rows in
+//   registers for the whole portion, so that a group costs one round of reductions (sixteen sums over sixteen lanes
+//   share their shuffles). Operands arrive in rounds by cp.async, two rounds ahead; products and sums are packed pairs of
+//   floats.
 // mx_delta_step: steps in which no sequence brings more than one token. A block owns (sequence, head): the state passes
 //   through registers once (a warp per group of value columns, a lane per four rows), reductions of sixteen columns
 //   share their shuffles, and the norm over the head's values, its weight and the gate follow in the same kernel.
@@ -30,7 +34,11 @@
 
 namespace {
 
-constexpr int DR_COLS = 16, DR_LANES = 8, DR_THREADS = DR_COLS * DR_LANES;
+constexpr int DR_COLS = 16, DR_LANES = 16, DR_THREADS = DR_COLS / 2 * DR_LANES;
+constexpr int DR_GROUP = 8;                  // tokens of a group
+constexpr int DR_STAGES = 3;                 // rounds of the scan in shared memory: one computed, two on their way
+// a group's numbers: T and P (a row per token), the fades from its start to each token and from each token to its end
+constexpr int DR_P = DR_GROUP * DR_GROUP, DR_FADE = 2 * DR_P, DR_END = DR_FADE + DR_GROUP, DR_COEF = DR_END + DR_GROUP;
 
 // ln(1 + e^x) without overflow on either side
 __device__ __forceinline__ float softplus_exact(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -180,11 +188,6 @@ __device__ __forceinline__ void copy16(float* smem, const float* global, bool li
     const int bytes = live ? 16 : 0;                         // nothing read: sixteen zero bytes
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(at), "l"(global), "r"(bytes));
 }
-__device__ __forceinline__ void copy4(float* smem, const float* global, bool live) {
-    const unsigned at = (unsigned)__cvta_generic_to_shared(smem);
-    const int bytes = live ? 4 : 0;
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;\n" ::"r"(at), "l"(global), "r"(bytes));
-}
 __device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;\n" ::: "memory"); }
 template <int LEFT>
 __device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(LEFT) : "memory"); }
@@ -194,165 +197,26 @@ struct DeltaParams {
     const float* beta;          // [tokens][heads]
     const float* decay;         // [tokens][heads], or [tokens][heads][dim]
     float* state;               // [slots][state_stride], S at state_offset as [heads][vdim][dim]
+    const int* tok_seq;
     const int* cu_q;
     const int* state_slots;
     float* out;                 // scan: [tokens][heads * vdim]
+    float* coef;                // scan: [groups][heads][DR_COEF]
+    float* decayed;             // scan, decays per channel: [3][tokens][heads][dim]: k, q decayed from the group's start, k to its end
+    float* group_decay;         // scan, decays per channel: [groups][heads][dim]
     long long state_stride, state_offset;
-    int channels, k_col, v_col, qk_heads, heads, dim, vdim;
+    int channels, k_col, v_col, qk_heads, heads, dim, vdim, n_tokens;
 };
 
-// ROWS rows of a column a lane (dim <= 8 * ROWS): the groups of four rows 4 (lane + 8 u), so that eight lanes' 16-byte
-// loads are one contiguous row
-template <int ROWS, int TOKENS, bool CHANNEL>
-struct ScanStage {
-    static constexpr int CH = DR_LANES * ROWS;
-    float k[TOKENS][CH], q[TOKENS][CH], g[CHANNEL ? TOKENS : 1][CHANNEL ? CH : 4], v[TOKENS][DR_COLS], beta[TOKENS], g1[TOKENS];
-};
+// The group that the token `local` tokens into a sequence's portion opens or belongs to: portions start groups of their own.
+__device__ __forceinline__ int group_of(int first, int seq, int local) { return (first + (DR_GROUP - 1) * seq) / DR_GROUP + local / DR_GROUP; }
 
-template <int ROWS, int TOKENS, bool CHANNEL>
-__global__ void __launch_bounds__(DR_THREADS)
-delta_scan_kernel(const DeltaParams p) {
-    using Stage = ScanStage<ROWS, TOKENS, CHANNEL>;
-    constexpr int CH = Stage::CH, R4 = ROWS / 4;
-    extern __shared__ __align__(16) unsigned char scan_smem[];
-    Stage* stages = reinterpret_cast<Stage*>(scan_smem);     // two rounds in flight
-    __shared__ float o_s[TOKENS][DR_LANES][DR_COLS];
-    pdl_trigger();
-    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * DR_COLS, tid = threadIdx.x;
-    const int t0 = p.cu_q[seq], t1 = p.cu_q[seq + 1];
-    if (t1 <= t0) {
-        // a padding sequence of a fixed-size batch, whose row bears its own number: defined output, no state
-        pdl_wait();
-        if (seq >= t0 && tid < DR_COLS && col0 + tid < p.vdim)
-            p.out[((size_t)seq * p.heads + head) * p.vdim + col0 + tid] = 0.f;
-        return;
-    }
-    const int lane = tid & (DR_LANES - 1), c = tid / DR_LANES, col = col0 + c;
-    const int qk_head = head / (p.heads / p.qk_heads);
-    const bool live_col = col < p.vdim;
-    float* s_base = p.state + (size_t)p.state_slots[seq] * p.state_stride + p.state_offset + ((size_t)head * p.vdim + col) * p.dim;
-    float4 S[R4];
-#pragma unroll
-    for (int u = 0; u < R4; ++u) {
-        const int r = 4 * (lane + DR_LANES * u);
-        S[u] = live_col && r < p.dim ? *reinterpret_cast<const float4*>(s_base + r) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    pdl_wait();
-    const float* qkv = after_wait(p.qkv);
-    const float* beta = after_wait(p.beta);
-    const float* decay = after_wait(p.decay);
-    auto fetch = [&](Stage& s, int base) {
-        for (int item = tid; item < TOKENS * (CH / 4); item += DR_THREADS) {
-            const int j = item / (CH / 4), r = (item % (CH / 4)) * 4, t = min(base + j, t1 - 1);
-            const bool live = base + j < t1 && r < p.dim;
-            const float* row = qkv + (size_t)t * p.channels + qk_head * p.dim + (r < p.dim ? r : 0);
-            copy16(&s.q[j][r], row, live);
-            copy16(&s.k[j][r], row + p.k_col, live);
-            if (CHANNEL) copy16(&s.g[CHANNEL ? j : 0][CHANNEL ? r : 0],
-                                decay + ((size_t)t * p.heads + head) * p.dim + (r < p.dim ? r : 0), live);
-        }
-        for (int item = tid; item < TOKENS * (DR_COLS / 4); item += DR_THREADS) {
-            const int j = item / (DR_COLS / 4), e = (item % (DR_COLS / 4)) * 4, t = min(base + j, t1 - 1);
-            const bool live = base + j < t1 && col0 + e < p.vdim;
-            copy16(&s.v[j][e], qkv + (size_t)t * p.channels + p.v_col + head * p.vdim + (col0 + e < p.vdim ? col0 + e : 0), live);
-        }
-        if (tid < TOKENS) {
-            const int t = min(base + tid, t1 - 1);
-            copy4(&s.beta[tid], beta + (size_t)t * p.heads + head, base + tid < t1);
-            if (!CHANNEL) copy4(&s.g1[tid], decay + (size_t)t * p.heads + head, base + tid < t1);
-        }
-        copies_commit();
-    };
-    struct Operands {
-        float4 k[R4], q[R4], g[CHANNEL ? R4 : 1];
-        float v, beta, g1;
-    };
-    auto read = [&](Operands& into, const Stage& s, int j) {
-#pragma unroll
-        for (int u = 0; u < R4; ++u) {
-            const int r = 4 * (lane + DR_LANES * u);
-            into.k[u] = *reinterpret_cast<const float4*>(&s.k[j][r]);
-            into.q[u] = *reinterpret_cast<const float4*>(&s.q[j][r]);
-            if (CHANNEL) into.g[CHANNEL ? u : 0] = *reinterpret_cast<const float4*>(&s.g[CHANNEL ? j : 0][CHANNEL ? r : 0]);
-        }
-        into.v = s.v[j][c];
-        into.beta = s.beta[j];
-        into.g1 = CHANNEL ? 1.f : s.g1[j];
-    };
-    auto advance = [&](const Operands& now, int j) {
-        float4 held = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (int u = 0; u < R4; ++u) {
-            const float4 g = CHANNEL ? now.g[CHANNEL ? u : 0] : make_float4(now.g1, now.g1, now.g1, now.g1);
-            S[u].x *= g.x; S[u].y *= g.y; S[u].z *= g.z; S[u].w *= g.w;
-            held.x = fmaf(S[u].x, now.k[u].x, held.x); held.y = fmaf(S[u].y, now.k[u].y, held.y);
-            held.z = fmaf(S[u].z, now.k[u].z, held.z); held.w = fmaf(S[u].w, now.k[u].w, held.w);
-        }
-        float sum = (held.x + held.y) + (held.z + held.w);
-#pragma unroll
-        for (int o = DR_LANES / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-        const float write = now.beta * (now.v - sum);
-        float4 read_out = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (int u = 0; u < R4; ++u) {
-            S[u].x = fmaf(now.k[u].x, write, S[u].x); S[u].y = fmaf(now.k[u].y, write, S[u].y);
-            S[u].z = fmaf(now.k[u].z, write, S[u].z); S[u].w = fmaf(now.k[u].w, write, S[u].w);
-            read_out.x = fmaf(S[u].x, now.q[u].x, read_out.x); read_out.y = fmaf(S[u].y, now.q[u].y, read_out.y);
-            read_out.z = fmaf(S[u].z, now.q[u].z, read_out.z); read_out.w = fmaf(S[u].w, now.q[u].w, read_out.w);
-        }
-        o_s[j][lane][c] = (read_out.x + read_out.y) + (read_out.z + read_out.w);
-    };
-    fetch(stages[0], t0);
-    int at = 0;
-    for (int base = t0; base < t1; base += TOKENS, at ^= 1) {
-        const int n_here = min(TOKENS, t1 - base);
-        if (base + TOKENS < t1) {
-            fetch(stages[at ^ 1], base + TOKENS);
-            copies_wait<1>();
-        } else {
-            copies_wait<0>();
-        }
-        __syncthreads();
-        const Stage& s = stages[at];
-        Operands even, odd;
-        read(even, s, 0);
-        for (int j = 0; j < n_here; j += 2) {
-            if (j + 1 < n_here) read(odd, s, j + 1);
-            advance(even, j);
-            if (j + 1 < n_here) {
-                if (j + 2 < n_here) read(even, s, j + 2);
-                advance(odd, j + 1);
-            }
-        }
-        __syncthreads();                                     // the round's shares are there, its operands are done with
-        for (int item = tid; item < n_here * DR_COLS; item += DR_THREADS) {
-            const int j = item / DR_COLS, e = item % DR_COLS;
-            float o = 0.f;
-#pragma unroll
-            for (int l = 0; l < DR_LANES; ++l) o += o_s[j][l][e];
-            if (col0 + e < p.vdim) p.out[((size_t)(base + j) * p.heads + head) * p.vdim + col0 + e] = o;
-        }
-    }
-#pragma unroll
-    for (int u = 0; u < R4; ++u) {
-        const int r = 4 * (lane + DR_LANES * u);
-        if (live_col && r < p.dim) *reinterpret_cast<float4*>(s_base + r) = S[u];
-    }
-}
-
-struct StepParams {
-    DeltaParams d;
-    const float* gate;          // rows gate_ld floats apart: [heads * vdim] logits
-    const float* weight;        // [vdim]
-    int gate_ld, out_ld, sigmoid_gate, true_vdim;
-    float eps, out_scale;
-};
-
-// N sums over a warp that share their shuffles: on return lane l holds the sum number l / (32 / N)
-template <int N>
+// N sums over groups of LANES neighbouring lanes that share their shuffles: on return lane l of a group holds the sum number
+// l / (LANES / N)
+template <int N, int LANES>
 __device__ __forceinline__ float shared_sums(float (&v)[N]) {
-    const int lane = threadIdx.x & 31;
-    int w = 16;
+    const int lane = threadIdx.x & (LANES - 1);
+    int w = LANES / 2;
 #pragma unroll
     for (int n = N; n > 1; n >>= 1, w >>= 1) {
         const bool upper = lane & w;
@@ -363,9 +227,379 @@ __device__ __forceinline__ float shared_sums(float (&v)[N]) {
         }
     }
     float sum = v[0];
+#pragma unroll
     for (; w > 0; w >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, w);
     return sum;
 }
+
+__device__ __forceinline__ float4 times(const float4& a, const float4& b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float dot4(const float4& a, const float4& b, float sum) {
+    return fmaf(a.w, b.w, fmaf(a.z, b.z, fmaf(a.y, b.y, fmaf(a.x, b.x, sum))));
+}
+
+// A warp per (group of tokens, head): what the tokens of a group do to one another, whatever the state.
+template <int NV, bool CHANNEL>
+__global__ void __launch_bounds__(128)
+delta_groups_kernel(const DeltaParams p) {
+    constexpr int N = DR_GROUP, PAIRS = N * (N - 1) / 2;     // k_i k_j for i > j, then q_i k_j for i >= j: N * N sums
+    static_assert(N * N == 64, "the sums of a group are two to a lane");
+    __shared__ float sums_s[4][N * N];
+    pdl_trigger();
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, head = blockIdx.y * 4 + warp, lane = threadIdx.x & 31;
+    const int seq = p.tok_seq[t];
+    if (seq < 0 || head >= p.heads) return;
+    const int first = p.cu_q[seq], local = t - first;
+    if (local % N) return;                                   // one warp per group: the one of its first token
+    const int n_here = min(N, p.cu_q[seq + 1] - t), group = group_of(first, seq, local);
+    pdl_wait();
+    const float* qkv = after_wait(p.qkv) + (head / (p.heads / p.qk_heads)) * p.dim;
+    const float* beta_in = after_wait(p.beta);
+    const float* decay = after_wait(p.decay);
+    // a token that is not there: nothing fades, nothing is written
+    const float my_beta = lane < n_here ? beta_in[(size_t)(t + lane) * p.heads + head] : 0.f;
+    const float my_decay = !CHANNEL && lane < n_here ? decay[(size_t)(t + lane) * p.heads + head] : 1.f;
+    float low[32] = {}, high[32] = {};                       // sums 0 .. 31 and 32 .. 63
+    auto add = [&](int index, float v) {
+        if (index < 32) low[index] += v; else high[index - 32] += v;
+    };
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+        const int r = 4 * lane + 128 * n;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), one = make_float4(1.f, 1.f, 1.f, 1.f);
+        float4 k[N], q[N], g[CHANNEL ? N : 1];
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const bool live = i < n_here && r < p.dim;
+            const float* row = qkv + (size_t)(t + i) * p.channels + r;
+            q[i] = live ? *reinterpret_cast<const float4*>(row) : zero;
+            k[i] = live ? *reinterpret_cast<const float4*>(row + p.k_col) : zero;
+            if (CHANNEL)
+                g[CHANNEL ? i : 0] = live ? *reinterpret_cast<const float4*>(decay + ((size_t)(t + i) * p.heads + head) * p.dim + r) : one;
+        }
+        const size_t plane = (size_t)p.n_tokens * p.heads * p.dim;
+        float* dst = p.decayed + ((size_t)t * p.heads + head) * p.dim + r;
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+            float4 w = k[j];                                 // the key of j as it has faded by token i
+            add(PAIRS + j * (j + 1) / 2 + j, dot4(q[j], w, 0.f));
+#pragma unroll
+            for (int i = j + 1; i < N; ++i) {
+                if (CHANNEL) w = times(w, g[CHANNEL ? i : 0]);
+                add(i * (i - 1) / 2 + j, dot4(k[i], w, 0.f));
+                add(PAIRS + i * (i + 1) / 2 + j, dot4(q[i], w, 0.f));
+            }
+            if (CHANNEL && j < n_here && r < p.dim)
+                *reinterpret_cast<float4*>(dst + 2 * plane + (size_t)j * p.heads * p.dim) = w;
+        }
+        if (CHANNEL && r < p.dim) {
+            float4 fade = one;
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                fade = times(fade, g[CHANNEL ? i : 0]);
+                if (i >= n_here) continue;
+                *reinterpret_cast<float4*>(dst + (size_t)i * p.heads * p.dim) = times(k[i], fade);
+                *reinterpret_cast<float4*>(dst + plane + (size_t)i * p.heads * p.dim) = times(q[i], fade);
+            }
+            *reinterpret_cast<float4*>(p.group_decay + ((size_t)group * p.heads + head) * p.dim + r) = fade;
+        }
+    }
+    float* sums = sums_s[warp];
+    sums[lane] = shared_sums<32, 32>(low);
+    sums[32 + lane] = shared_sums<32, 32>(high);
+    __syncwarp();
+    float decays[N], betas[N];                               // decays: ones where each channel has its own
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        decays[i] = __shfl_sync(0xffffffffu, my_decay, i);
+        betas[i] = __shfl_sync(0xffffffffu, my_beta, i);
+    }
+    if (lane >= N) return;
+    // lane j: column j of T and of P. u = T (v - S^T k, decayed) solves u_i = beta_i (v_i - .. - sum_(j<i) (k_i k_j) u_j)
+    float* coef = p.coef + ((size_t)group * p.heads + head) * DR_COEF;
+    float T[N];                                              // of rows lane .. N - 1
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        float sum = 0.f, left = 1.f;
+#pragma unroll
+        for (int m = i - 1; m >= 0; --m) {
+            left *= decays[m + 1];                           // what is left of token m's key at token i
+            if (m >= lane) sum = fmaf(sums[i * (i - 1) / 2 + m] * left, T[m], sum);
+        }
+        T[i] = i < lane ? 0.f : (i == lane ? betas[i] : -betas[i] * sum);
+        coef[i * N + lane] = T[i];
+    }
+    float left = 1.f, fade = 1.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        if (i > lane) left *= decays[i];
+        coef[DR_P + i * N + lane] = i >= lane ? sums[PAIRS + i * (i + 1) / 2 + min(lane, i)] * left : 0.f;
+        fade *= decays[i];
+        if (i == lane) coef[DR_FADE + i] = fade;
+    }
+    coef[DR_END + lane] = left;
+}
+
+// A round's operands. Sixteen lanes share two value columns, R4 groups of four rows a lane (dim <= 64 * R4): the rows
+// 4 (lane + 16 u), so that sixteen lanes' 16-byte loads are one contiguous row.
+template <int R4, int TOKENS, bool CHANNEL>
+struct ScanStage {
+    static constexpr int CH = 4 * DR_LANES * R4, GROUPS = TOKENS / DR_GROUP;
+    float k[TOKENS][CH], q[TOKENS][CH], k_end[CHANNEL ? TOKENS : 1][CHANNEL ? CH : 4], fade[CHANNEL ? GROUPS : 1][CHANNEL ? CH : 4];
+    float v[TOKENS][DR_COLS], coef[GROUPS][DR_COEF];
+};
+
+// Pairs of floats as the packed operations take them.
+using Pair = unsigned long long;
+__device__ __forceinline__ Pair fma2(Pair a, Pair b, Pair c) {
+    Pair d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ Pair mul2(Pair a, Pair b) {
+    Pair d;
+    asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ Pair both(float v) {
+    Pair d;
+    asm("mov.b64 %0, {%1, %1};\n" : "=l"(d) : "f"(v));
+    return d;
+}
+__device__ __forceinline__ float sum2(Pair a) {
+    float x, y;
+    asm("mov.b64 {%0, %1}, %2;\n" : "=f"(x), "=f"(y) : "l"(a));
+    return x + y;
+}
+struct Quad { Pair a, b; };                                  // four neighbouring rows
+__device__ __forceinline__ Quad load_quad(const float* p) {
+    const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
+    return {v.x, v.y};
+}
+// The same from shared memory, set out where it stands: the compiler moves no such load towards its use (with decays per
+// channel it otherwise loads quad by quad and waits for each; with one per head it does better by itself).
+__device__ __forceinline__ Quad ask_quad(const float* p) {
+    Quad v;
+    asm volatile("ld.shared.v2.b64 {%0, %1}, [%2];\n" : "=l"(v.a), "=l"(v.b) : "r"((unsigned)__cvta_generic_to_shared(p)) : "memory");
+    return v;
+}
+
+template <int R4, int TOKENS, bool CHANNEL>
+__global__ void __launch_bounds__(DR_THREADS)
+delta_scan_kernel(const DeltaParams p) {
+    using Stage = ScanStage<R4, TOKENS, CHANNEL>;
+    constexpr int CH = Stage::CH, ROW_THREADS = CH / 4, ROWS = DR_THREADS / ROW_THREADS;
+    static_assert(DR_THREADS % ROW_THREADS == 0 && TOKENS % ROWS == 0, "a round's rows fill whole passes");
+    extern __shared__ __align__(16) unsigned char scan_smem[];
+    Stage* stages = reinterpret_cast<Stage*>(scan_smem);     // DR_STAGES rounds
+    pdl_trigger();
+    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * DR_COLS, tid = threadIdx.x;
+    const int t0 = p.cu_q[seq], t1 = p.cu_q[seq + 1];
+    if (t1 <= t0) {
+        // a padding sequence of a fixed-size batch, whose row bears its own number: defined output, no state
+        pdl_wait();
+        if (seq >= t0 && tid < DR_COLS && col0 + tid < p.vdim)
+            p.out[((size_t)seq * p.heads + head) * p.vdim + col0 + tid] = 0.f;
+        return;
+    }
+    const int lane = tid & (DR_LANES - 1), c = 2 * (tid / DR_LANES), col = col0 + c;
+    const int group0 = group_of(t0, seq, 0);
+    float* s_base = p.state + (size_t)p.state_slots[seq] * p.state_stride + p.state_offset + ((size_t)head * p.vdim + col) * p.dim;
+    Quad S[2][R4];
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+        for (int u = 0; u < R4; ++u) {
+            const int r = 4 * (lane + DR_LANES * u);
+            S[x][u] = col + x < p.vdim && r < p.dim ? load_quad(s_base + (size_t)x * p.dim + r) : Quad{0, 0};
+        }
+    if (p.dim < CH) {
+        // the rows that no head has stay zero in every round
+        for (int i = tid; i < (int)(DR_STAGES * sizeof(Stage) / 16); i += DR_THREADS)
+            reinterpret_cast<float4*>(scan_smem)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        __syncthreads();
+    }
+    pdl_wait();
+    // a thread copies the same four rows of every ROWS-th token
+    const int row_j = tid / ROW_THREADS, r0 = (tid % ROW_THREADS) * 4;
+    const bool copies = r0 < p.dim;
+    const size_t plane = (size_t)p.n_tokens * p.heads * p.dim, row_stride = CHANNEL ? (size_t)p.heads * p.dim : (size_t)p.channels;
+    const float* k_from = CHANNEL ? after_wait(p.decayed) + ((size_t)t0 * p.heads + head) * p.dim + r0
+                                  : after_wait(p.qkv) + (size_t)t0 * p.channels + p.k_col + (head / (p.heads / p.qk_heads)) * p.dim + r0;
+    const float* q_from = CHANNEL ? k_from + plane : k_from - p.k_col;
+    const float* v_from = after_wait(p.qkv) + (size_t)t0 * p.channels + p.v_col + head * p.vdim + col0;
+    const float* coef = after_wait(p.coef) + ((size_t)group0 * p.heads + head) * DR_COEF;
+    const float* group_decay = after_wait(p.group_decay) + ((size_t)group0 * p.heads + head) * p.dim;
+    const int n = t1 - t0;
+    auto fetch = [&](Stage& s, int base) {                   // tokens base .. of the portion; an empty group when there are none
+        if (base < n) {
+            const bool whole = base + TOKENS <= n;
+            if (copies) {
+                const size_t at = (size_t)(base + row_j) * row_stride;
+                const float *k_at = k_from + at, *q_at = q_from + at;
+#pragma unroll
+                for (int j = 0; j < TOKENS; j += ROWS) {
+                    const bool live = whole || base + row_j + j < n;
+                    const float *k = live ? k_at : k_from, *q = live ? q_at : q_from;
+                    copy16(&s.k[row_j + j][r0], k, live);
+                    copy16(&s.q[row_j + j][r0], q, live);
+                    if (CHANNEL) copy16(&s.k_end[CHANNEL ? row_j + j : 0][CHANNEL ? r0 : 0], k + 2 * plane, live);
+                    k_at += ROWS * row_stride;
+                    q_at += ROWS * row_stride;
+                }
+            }
+            if (tid < TOKENS * (DR_COLS / 4)) {
+                const int j = tid / (DR_COLS / 4), e = (tid % (DR_COLS / 4)) * 4;
+                const bool live = base + j < n && col0 + e < p.vdim;
+                copy16(&s.v[j][e], live ? v_from + (size_t)(base + j) * p.channels + e : v_from, live);
+            }
+            const int group = base / DR_GROUP, groups = (n - base + DR_GROUP - 1) / DR_GROUP;
+#pragma unroll
+            for (int g = 0; g < Stage::GROUPS; ++g) {
+                if (tid < DR_COEF / 4)
+                    copy16(&s.coef[g][4 * tid], coef + (size_t)(group + (g < groups ? g : 0)) * p.heads * DR_COEF + 4 * tid, g < groups);
+                if (CHANNEL && row_j == (g + 1) % ROWS && copies)
+                    copy16(&s.fade[CHANNEL ? g : 0][CHANNEL ? r0 : 0],
+                           group_decay + (size_t)(group + (g < groups ? g : 0)) * p.heads * p.dim + r0, g < groups);
+            }
+        }
+        copies_commit();
+    };
+    // the one of the group's sums that a lane ends up with: token own_i, column own_x
+    const int own_i = lane >> 1, own_x = lane & 1;
+    const bool writes = col + own_x < p.vdim;
+    const size_t out_stride = (size_t)p.heads * p.vdim;
+    float* out = p.out + ((size_t)(t0 + own_i) * p.heads + head) * p.vdim + col + own_x;
+    auto advance = [&](const Stage& s, int g, int t) {
+        const int j0 = g * DR_GROUP;
+        const float* numbers = s.coef[g];
+        Pair pairs[2 * DR_GROUP];
+        float sums[2 * DR_GROUP];
+        Quad k[DR_GROUP][R4], q[DR_GROUP][R4];
+        auto ask = [&](Quad (&into)[DR_GROUP][R4], const float (*rows)[CH]) {
+#pragma unroll
+            for (int i = 0; i < DR_GROUP; ++i)
+#pragma unroll
+                for (int u = 0; u < R4; ++u) {
+                    const float* at = &rows[j0 + i][4 * (lane + DR_LANES * u)];
+                    into[i][u] = CHANNEL ? ask_quad(at) : load_quad(at);
+                }
+        };
+        auto contract = [&](const Quad (&m)[DR_GROUP][R4]) {
+#pragma unroll
+            for (int i = 0; i < 2 * DR_GROUP; ++i) pairs[i] = 0;
+#pragma unroll
+            for (int u = 0; u < R4; ++u) {
+#pragma unroll
+                for (int i = 0; i < DR_GROUP; ++i) {
+                    pairs[2 * i] = fma2(S[0][u].a, m[i][u].a, pairs[2 * i]);
+                    pairs[2 * i + 1] = fma2(S[1][u].a, m[i][u].a, pairs[2 * i + 1]);
+                }
+#pragma unroll
+                for (int i = 0; i < DR_GROUP; ++i) {
+                    pairs[2 * i] = fma2(S[0][u].b, m[i][u].b, pairs[2 * i]);
+                    pairs[2 * i + 1] = fma2(S[1][u].b, m[i][u].b, pairs[2 * i + 1]);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 2 * DR_GROUP; ++i) sums[i] = sum2(pairs[i]);
+        };
+        ask(k, s.k);
+        const float my_fade = CHANNEL ? 1.f : numbers[DR_FADE + own_i];
+        const float my_v = s.v[j0 + own_i][c + own_x];
+        ask(q, s.q);
+        contract(k);
+        // v - S^T k of the lane's own token and column, then its row of T times those of the group
+        const float mine = fmaf(-my_fade, shared_sums<2 * DR_GROUP, DR_LANES>(sums), my_v);
+        contract(q);
+        if constexpr (CHANNEL) ask(k, s.k_end);
+        float write[2] = {0.f, 0.f};
+#pragma unroll
+        for (int j = 0; j < DR_GROUP; j += 4) {
+            const float4 row = *reinterpret_cast<const float4*>(&numbers[own_i * DR_GROUP + j]);
+            write[0] = fmaf(row.x, __shfl_sync(0xffffffffu, mine, 2 * j + own_x, DR_LANES), write[0]);
+            write[1] = fmaf(row.y, __shfl_sync(0xffffffffu, mine, 2 * j + 2 + own_x, DR_LANES), write[1]);
+            write[0] = fmaf(row.z, __shfl_sync(0xffffffffu, mine, 2 * j + 4 + own_x, DR_LANES), write[0]);
+            write[1] = fmaf(row.w, __shfl_sync(0xffffffffu, mine, 2 * j + 6 + own_x, DR_LANES), write[1]);
+        }
+        const float my_write = write[0] + write[1];
+        float w[DR_GROUP][2];
+#pragma unroll
+        for (int i = 0; i < DR_GROUP; ++i) {
+            w[i][0] = __shfl_sync(0xffffffffu, my_write, 2 * i, DR_LANES);
+            w[i][1] = __shfl_sync(0xffffffffu, my_write, 2 * i + 1, DR_LANES);
+        }
+        const float my_seen = shared_sums<2 * DR_GROUP, DR_LANES>(sums);
+        // o = S^T q + P u
+        float o[2] = {my_fade * my_seen, 0.f};
+#pragma unroll
+        for (int j = 0; j < DR_GROUP; j += 4) {
+            const float4 row = *reinterpret_cast<const float4*>(&numbers[DR_P + own_i * DR_GROUP + j]);
+            o[0] = fmaf(row.x, own_x ? w[j][1] : w[j][0], o[0]);
+            o[1] = fmaf(row.y, own_x ? w[j + 1][1] : w[j + 1][0], o[1]);
+            o[0] = fmaf(row.z, own_x ? w[j + 2][1] : w[j + 2][0], o[0]);
+            o[1] = fmaf(row.w, own_x ? w[j + 3][1] : w[j + 3][0], o[1]);
+        }
+        if (writes && t + own_i < n) out[(size_t)t * out_stride] = o[0] + o[1];
+        // the state at the group's end
+        if (!CHANNEL) {
+            const Pair fade = both(numbers[DR_FADE + DR_GROUP - 1]);
+#pragma unroll
+            for (int i = 0; i < DR_GROUP; i += 4) {
+                const float4 end = *reinterpret_cast<const float4*>(&numbers[DR_END + i]);
+                w[i][0] *= end.x; w[i][1] *= end.x; w[i + 1][0] *= end.y; w[i + 1][1] *= end.y;
+                w[i + 2][0] *= end.z; w[i + 2][1] *= end.z; w[i + 3][0] *= end.w; w[i + 3][1] *= end.w;
+            }
+#pragma unroll
+            for (int x = 0; x < 2; ++x)
+#pragma unroll
+                for (int u = 0; u < R4; ++u) S[x][u] = {mul2(S[x][u].a, fade), mul2(S[x][u].b, fade)};
+        } else {
+#pragma unroll
+            for (int u = 0; u < R4; ++u) {
+                const Quad f = load_quad(&s.fade[CHANNEL ? g : 0][CHANNEL ? 4 * (lane + DR_LANES * u) : 0]);
+#pragma unroll
+                for (int x = 0; x < 2; ++x) S[x][u] = {mul2(S[x][u].a, f.a), mul2(S[x][u].b, f.b)};
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < DR_GROUP; ++i) {
+            const Pair w0 = both(w[i][0]), w1 = both(w[i][1]);
+#pragma unroll
+            for (int u = 0; u < R4; ++u) {
+                const Quad e = k[i][u];
+                S[0][u] = {fma2(e.a, w0, S[0][u].a), fma2(e.b, w0, S[0][u].b)};
+                S[1][u] = {fma2(e.a, w1, S[1][u].a), fma2(e.b, w1, S[1][u].b)};
+            }
+        }
+    };
+    fetch(stages[0], 0);
+    fetch(stages[1], TOKENS);
+    int at = 0;
+    for (int base = 0; base < n; base += TOKENS) {
+        copies_wait<1>();
+        __syncthreads();                                     // the round is there, the one before it is done with
+        fetch(stages[at == 0 ? DR_STAGES - 1 : at - 1], base + 2 * TOKENS);
+        const int groups = min(Stage::GROUPS, (n - base + DR_GROUP - 1) / DR_GROUP);
+        for (int g = 0; g < groups; ++g) advance(stages[at], g, base + g * DR_GROUP);
+        at = at == DR_STAGES - 1 ? 0 : at + 1;
+    }
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+        for (int u = 0; u < R4; ++u) {
+            const int r = 4 * (lane + DR_LANES * u);
+            if (col + x < p.vdim && r < p.dim)
+                *reinterpret_cast<ulonglong2*>(s_base + (size_t)x * p.dim + r) = make_ulonglong2(S[x][u].a, S[x][u].b);
+        }
+}
+
+struct StepParams {
+    DeltaParams d;
+    const float* gate;          // rows gate_ld floats apart: [heads * vdim] logits
+    const float* weight;        // [vdim]
+    int gate_ld, out_ld, sigmoid_gate, true_vdim;
+    float eps, out_scale;
+};
 
 template <typename T, int NV, bool CHANNEL>
 __global__ void __launch_bounds__(256)
@@ -434,7 +668,7 @@ delta_step_kernel(const StepParams sp, T* __restrict__ out) {
                 seen[x] += fmaf(s.x, q[n].x, s.y * q[n].y) + fmaf(s.z, q[n].z, s.w * q[n].w);
             }
         }
-        const float sum_k = shared_sums<COLS>(held), sum_q = shared_sums<COLS>(seen);
+        const float sum_k = shared_sums<COLS, 32>(held), sum_q = shared_sums<COLS, 32>(seen);
         const int mine = e0 + lane / PER;
         const float write = mine < p.vdim ? beta * (v_row[mine] - sum_k) : 0.f;
         // S^T q after the write: what the forgetting state gives plus the write times k . q
@@ -473,27 +707,29 @@ void launch_prepare(const PrepareParams& p, cudaStream_t stream) {
         mx_launch_chained(delta_prepare_kernel<TAPS, 8, NV>, dim3((p.n_tokens + 7) / 8, (items + 3) / 4), dim3(128), 0, stream, p);
 }
 
-template <int ROWS, int TOKENS, bool CHANNEL>
+template <int R4, int TOKENS, bool CHANNEL>
 int launch_scan(const DeltaParams& p, int n_seqs, cudaStream_t stream) {
-    constexpr size_t smem = 2 * sizeof(ScanStage<ROWS, TOKENS, CHANNEL>);
+    constexpr size_t smem = DR_STAGES * sizeof(ScanStage<R4, TOKENS, CHANNEL>);
     static bool ready = false;
     if (!ready) {
-        if (cudaFuncSetAttribute(delta_scan_kernel<ROWS, TOKENS, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        if (cudaFuncSetAttribute(delta_scan_kernel<R4, TOKENS, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)smem) != cudaSuccess)
             MX_REFUSE("delta rule: cannot reserve %zu bytes of shared memory", smem);
         ready = true;
     }
-    mx_launch_chained(delta_scan_kernel<ROWS, TOKENS, CHANNEL>, dim3(n_seqs, p.heads, (p.vdim + DR_COLS - 1) / DR_COLS),
+    const dim3 grid(p.n_tokens, (p.heads + 3) / 4);
+    if (p.dim <= 128) mx_launch_chained(delta_groups_kernel<1, CHANNEL>, grid, dim3(128), 0, stream, p);
+    else mx_launch_chained(delta_groups_kernel<2, CHANNEL>, grid, dim3(128), 0, stream, p);
+    mx_launch_chained(delta_scan_kernel<R4, TOKENS, CHANNEL>, dim3(n_seqs, p.heads, (p.vdim + DR_COLS - 1) / DR_COLS),
                       dim3(DR_THREADS), smem, stream, p);
     return mx_launch_status();
 }
 
 template <bool CHANNEL>
 int pick_scan(const DeltaParams& p, int n_seqs, cudaStream_t stream) {
-    if (p.dim <= 32) return launch_scan<4, 16, CHANNEL>(p, n_seqs, stream);
-    if (p.dim <= 64) return launch_scan<8, 16, CHANNEL>(p, n_seqs, stream);
-    if (p.dim <= 128) return launch_scan<16, 16, CHANNEL>(p, n_seqs, stream);
-    return launch_scan<32, 8, CHANNEL>(p, n_seqs, stream);
+    if (p.dim <= 64) return launch_scan<1, 16, CHANNEL>(p, n_seqs, stream);
+    if (p.dim <= 128) return launch_scan<2, 16, CHANNEL>(p, n_seqs, stream);
+    return launch_scan<4, 8, CHANNEL>(p, n_seqs, stream);
 }
 
 const char* delta_sizes(int qk_heads, int heads, int dim, int vdim) {
@@ -544,27 +780,39 @@ extern "C" int mx_delta_decay(const float* low, int low_ld, const float* a2, con
 }
 
 static int delta_params(DeltaParams& p, const float* qkv, const float* beta, const float* decay, float* state,
-                        long long state_stride, long long state_offset, const int* cu_q, const int* state_slots, float* out,
+                        long long state_stride, long long state_offset, const int* cu_q, const int* state_slots,
                         int qk_heads, int heads, int dim, int vdim) {
     if (const char* what = delta_sizes(qk_heads, heads, dim, vdim)) MX_REFUSE("delta rule: %s: %d of %d, %d of %d", what, qk_heads, dim, heads, vdim);
     if (state_stride % 4 || state_offset % 4 || state_stride < state_offset + (long long)heads * dim * vdim)
         MX_REFUSE("delta rule: a state of %lld floats from %lld is too short", state_stride, state_offset);
     if (((uintptr_t)qkv | (uintptr_t)decay | (uintptr_t)state) % 16) MX_REFUSE("delta rule: unaligned operands");
-    p.qkv = qkv; p.beta = beta; p.decay = decay; p.state = state; p.cu_q = cu_q; p.state_slots = state_slots; p.out = out;
-    p.state_stride = state_stride; p.state_offset = state_offset; p.channels = 2 * qk_heads * dim + heads * vdim;
+    p.qkv = qkv; p.beta = beta; p.decay = decay; p.state = state; p.cu_q = cu_q; p.state_slots = state_slots;
+    p.tok_seq = nullptr; p.out = p.coef = p.decayed = p.group_decay = nullptr; p.n_tokens = 0; p.state_stride = state_stride; p.state_offset = state_offset; p.channels = 2 * qk_heads * dim + heads * vdim;
     p.k_col = qk_heads * dim; p.v_col = 2 * qk_heads * dim; p.qk_heads = qk_heads; p.heads = heads; p.dim = dim; p.vdim = vdim;
     return MX_OK;
 }
 
+// How many floats mx_delta_scan wants as scratch.
+extern "C" long long mx_delta_scan_scratch(int per_channel, int n_tokens, int n_seqs, int heads, int dim) {
+    const long long groups = (n_tokens + (long long)(DR_GROUP - 1) * n_seqs) / DR_GROUP + 1;
+    return groups * heads * DR_COEF + (per_channel ? (3LL * n_tokens + groups) * heads * dim : 0);
+}
+
 // `per_channel`: decay is [tokens][heads][dim] instead of [tokens][heads]
 extern "C" int mx_delta_scan(const float* qkv, const float* beta, const float* decay, int per_channel, float* state,
-                             long long state_stride, long long state_offset, const int* cu_q, const int* state_slots,
-                             float* out, int n_seqs, int qk_heads, int heads, int dim, int vdim, cudaStream_t stream) {
-    if (n_seqs <= 0) return MX_OK;
+                             long long state_stride, long long state_offset, const int* tok_seq, const int* cu_q,
+                             const int* state_slots, float* scratch, float* out, int n_tokens, int n_seqs, int qk_heads,
+                             int heads, int dim, int vdim, cudaStream_t stream) {
+    if (n_seqs <= 0 || n_tokens <= 0) return MX_OK;
     DeltaParams p;
-    const int rc = delta_params(p, qkv, beta, decay, state, state_stride, state_offset, cu_q, state_slots, out, qk_heads, heads,
-                                dim, vdim);
+    const int rc = delta_params(p, qkv, beta, decay, state, state_stride, state_offset, cu_q, state_slots, qk_heads, heads, dim,
+                                vdim);
     if (rc != MX_OK) return rc;
+    if ((uintptr_t)scratch % 16) MX_REFUSE("delta rule: unaligned scratch memory");
+    const long long groups = (n_tokens + (long long)(DR_GROUP - 1) * n_seqs) / DR_GROUP + 1;
+    p.tok_seq = tok_seq; p.out = out; p.n_tokens = n_tokens; p.coef = scratch;
+    p.group_decay = scratch + groups * heads * DR_COEF;
+    p.decayed = p.group_decay + groups * heads * dim;
     return per_channel ? pick_scan<true>(p, n_seqs, stream) : pick_scan<false>(p, n_seqs, stream);
 }
 
@@ -577,8 +825,8 @@ extern "C" int mx_delta_step(const float* qkv, const float* beta, const float* d
                              int true_vdim, cudaStream_t stream) {
     if (n_seqs <= 0) return MX_OK;
     StepParams sp;
-    const int rc = delta_params(sp.d, qkv, beta, decay, state, state_stride, state_offset, cu_q, state_slots, nullptr, qk_heads,
-                                heads, dim, vdim);
+    const int rc = delta_params(sp.d, qkv, beta, decay, state, state_stride, state_offset, cu_q, state_slots, qk_heads, heads,
+                                dim, vdim);
     if (rc != MX_OK) return rc;
     if (true_vdim <= 0 || true_vdim > vdim || vdim > 12 * 1024) MX_REFUSE("delta rule: heads of %d values in %d", true_vdim, vdim);
     sp.gate = gate; sp.weight = weight; sp.gate_ld = gate_ld; sp.out_ld = out_ld; sp.sigmoid_gate = sigmoid_gate;

@@ -1145,18 +1145,20 @@ def _delta_operands(qkv, beta, decay, state, state_offset, qk_heads, heads, dim,
 
 
 def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, state_offset: int,
-               cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor, qk_heads: int, heads: int,
-               dim: int, vdim: int) -> None:
+               tok_seq: torch.Tensor, cu_q: torch.Tensor, state_slots: torch.Tensor, n_seqs: int, out: torch.Tensor,
+               qk_heads: int, heads: int, dim: int, vdim: int) -> None:
     """``S <- g S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q`` over every sequence's tokens in order, from and to S
     ([heads, vdim, dim] at ``state_offset`` of a sequence's ``state`` vector). ``decay`` [tokens, heads] or, one per key
     channel, [tokens, heads, dim]; ``out`` float32 [tokens, heads * vdim]."""
     n, per_channel = _delta_operands(qkv, beta, decay, state, state_offset, qk_heads, heads, dim, vdim)
     _need(out, "out", torch.float32)
     assert tuple(out.shape) == (n, heads * vdim)
+    scratch = torch.empty(int(library().mx_delta_scan_scratch(per_channel, n, n_seqs, heads, dim)), dtype=torch.float32,
+                          device=qkv.device)
     check(library().mx_delta_scan(_ptr(qkv), _ptr(beta), _ptr(decay), per_channel, _ptr(state), state.stride(0),
-                                  int(state_offset), _ptr(cu_q), _ptr(state_slots), _ptr(out), n_seqs, qk_heads, heads, dim,
-                                  vdim, _stream()), "delta_scan")
-    _launched()
+                                  int(state_offset), _ptr(tok_seq), _ptr(cu_q), _ptr(state_slots), _ptr(scratch), _ptr(out), n,
+                                  n_seqs, qk_heads, heads, dim, vdim, _stream()), "delta_scan")
+    _launched(2)
 
 
 def delta_step(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, state_offset: int,

@@ -81,7 +81,8 @@ _SIGNATURES: dict[str, tuple[list, object]] = {
     "mx_norm_gate_rows": ([P, P, I, P, F, P, I, I, I, I, I, P], I),
     "mx_delta_prepare": ([P, I, I, I, P, I, P, P, P, L, P, P, P, P, P, P, I, I, I, I, I, F, F, P], I),
     "mx_delta_decay": ([P, I, P, P, P, P, I, I, I, I, P], I),
-    "mx_delta_scan": ([P, P, P, I, P, L, L, P, P, P, I, I, I, I, I, P], I),
+    "mx_delta_scan_scratch": ([I, I, I, I, I], L),
+    "mx_delta_scan": ([P, P, P, I, P, L, L, P, P, P, P, P, I, I, I, I, I, I, P], I),
     "mx_delta_step": ([P, P, P, I, P, L, L, P, P, P, I, I, P, F, F, P, I, I, I, I, I, I, I, I, P], I),
     "mx_moe_route": ([P, I, I, P, I, I, I, I, I, F, I, P, P, P, P, I, P], I),
     "mx_moe_route_softmax": ([P, I, I, P, I, I, I, I, I, I, P, P, P, P, P, P, I, P], I),

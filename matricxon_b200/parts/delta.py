@@ -8,7 +8,7 @@ continues from it and leaves it for the next one, so a sequence may be cut anywh
 
 One fused product gives float rows ``[q | k | v | gate | decay | beta]`` (the low-rank maps' first products in the places of
 gate and decay); a kernel convolves, activates and normalises them and forms the steps, another the decays per channel from
-float operands. Portions run through the recurrence token by token with the state in registers; steps of one token a sequence
+float operands. Portions run through the recurrence in groups of eight tokens with the state in registers; steps of one token a sequence
 have a kernel of their own that also ends the mixer (norm, weight, gate). Everything between the products is float in
 both dtypes; of the low-rank maps the decay's second product is float too, the gate's runs in the runtime dtype.
 
@@ -160,7 +160,7 @@ class DeltaRule(BranchMixer):
             return
         kernels.conv_state_update(proj, None, state, ctx.cu_q, ctx.state_slots, ctx.n_seqs, self.channels, self.taps)
         o = torch.empty((n, heads * vdim), dtype=torch.float32, device=device)
-        kernels.delta_scan(qkv, beta, decay, state, offset, ctx.cu_q, ctx.state_slots, ctx.n_seqs, o, s.num_kv_heads, heads,
-                           dim, vdim)
+        kernels.delta_scan(qkv, beta, decay, state, offset, ctx.tok_seq, ctx.cu_q, ctx.state_slots, ctx.n_seqs, o,
+                           s.num_kv_heads, heads, dim, vdim)
         kernels.gla_norm_gate(o, gate, self.norm_weight, s.eps, out, heads, vdim, sigmoid_gate=sigmoid, out_scale=scale,
                               true_vdim=s.value_dim)
