@@ -23,6 +23,8 @@ models (rotated windowed attention, routed experts through the same grouped prod
 models (attention in every layer with normalised queries and keys, routed experts, norms on the branches).
 ``--compare seredra`` does the same for the Seredra architecture beside Parunex, the closest of the engine's other models
 (attention and recurrent layers in turn, sigmoid-routed experts through the same grouped products).
+``--compare palelix`` does the same for the Palelix architecture beside Seredra, the closest of the engine's other models
+(attention beside a recurrence, linear attention with a constant decay, short convolutions, routed experts).
 """
 
 from __future__ import annotations
@@ -454,6 +456,28 @@ def seredra_config(size: dict) -> dict:
             "norm": {"eps": 1e-5}, "layers": layers}
 
 
+def palelix_config(size: dict) -> dict:
+    """Six layers of which the second and third run twice (eight layer runs): attention beside a delta rule with a decay per
+    key channel, lightning attention, and the delta rule with a decay per head, 128-wide heads everywhere (the attention's
+    over 4 KV heads, half as many q/k heads as value heads in the delta layers); the first layer with a dense gated
+    feed-forward, the others with eight clamped experts of half that width in four groups, two per token."""
+    w, h = size["width"], size["width"] // 128
+    dense = {"kind": "dense", "ff": size["ff"]}
+    routed = {"kind": "moe", "expert": {"ff": size["ff"] // 2, "limit": 7.0},
+              "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}}
+    parallel = {"type": "parallel",
+                "mixer": {"left": {"heads": h, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                   "rot": {"base": 1000000.0, "dims": 64}}, "left_scale": 1.0,
+                          "right": {"heads": h, "kv_heads": h, "dim": 128, "vdim": 128, "conv": 4}, "right_scale": 1.0}}
+    lightning = {"type": "lightning",
+                 "mixer": {"heads": h, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 3.0 * i / h) for i in range(h)]}}
+    delta = {"type": "delta", "mixer": {"heads": h, "kv_heads": h // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    order = [parallel, lightning, delta, parallel, lightning, delta]
+    layers = [dict(layer, mlp=dense if i == 0 else routed) for i, layer in enumerate(order)]
+    return {"architecture": "Palelix", "vocab": COMPARE_VOCAB, "width": w, "norm": {"eps": 1e-6},
+            "loop": {"start": 1, "stop": 3, "times": 2}, "layers": layers}
+
+
 def starcoder2_like(size: dict) -> dict:
     return dict(STARCODER2_3B, num_hidden_layers=COMPARE_LAYERS, hidden_size=size["width"],
                 num_attention_heads=size["width"] // 128, num_key_value_heads=4, head_dim=128,
@@ -551,7 +575,9 @@ def compare_designs(args) -> int:
     clocks.start()
     sizes = [s for s in args.compare_sizes.split(",") if s]
     batches = [int(b) for b in args.compare_batches.split(",")]
-    if args.compare == "seredra":
+    if args.compare == "palelix":
+        designs = (("palelix", palelix_config), ("seredra", seredra_config))
+    elif args.compare == "seredra":
         designs = (("seredra", seredra_config), ("parunex", parunex_config))
     elif args.compare == "kefasun":
         designs = (("kefasun", kefasun_config), ("bafusun", bafusun_config))
@@ -598,10 +624,11 @@ def main() -> int:
                         help="leave out the 7B and 15B workloads through the scheduler")
     parser.add_argument("--no-graphs", action="store_true",
                         help="launch every kernel of a decode step by itself (for profilers)")
-    parser.add_argument("--compare", choices=["busatar", "parunex", "bafusun", "kefasun", "seredra"], default=None,
+    parser.add_argument("--compare", choices=["busatar", "parunex", "bafusun", "kefasun", "seredra", "palelix"],
+                        default=None,
                         help="instead of the headline workload: Busatar beside StarCoder2, Parunex beside Busatar, "
-                             "Bafusun beside Parunex, Kefasun beside Bafusun, or Seredra beside Parunex, at equal "
-                             "layer sizes (prefill and decode throughput at a few sizes)")
+                             "Bafusun beside Parunex, Kefasun beside Bafusun, Seredra beside Parunex, or Palelix beside "
+                             "Seredra, at equal layer sizes (prefill and decode throughput at a few sizes)")
     parser.add_argument("--compare-only", default=None,
                         help="with --compare: measure only this one of the two designs (for profilers)")
     parser.add_argument("--compare-sizes", default="w1024,w2048")
