@@ -474,43 +474,54 @@ delta_scan_kernel(const DeltaParams p) {
         const float* numbers = s.coef[g];
         Pair pairs[2 * DR_GROUP];
         float sums[2 * DR_GROUP];
-        Quad k[DR_GROUP][R4], q[DR_GROUP][R4];
+        Quad k[DR_GROUP][R4];
         auto ask = [&](Quad (&into)[DR_GROUP][R4], const float (*rows)[CH]) {
 #pragma unroll
             for (int i = 0; i < DR_GROUP; ++i)
 #pragma unroll
-                for (int u = 0; u < R4; ++u) {
-                    const float* at = &rows[j0 + i][4 * (lane + DR_LANES * u)];
-                    into[i][u] = CHANNEL ? ask_quad(at) : load_quad(at);
-                }
+                for (int u = 0; u < R4; ++u) into[i][u] = ask_quad(&rows[j0 + i][4 * (lane + DR_LANES * u)]);
         };
-        auto contract = [&](const Quad (&m)[DR_GROUP][R4]) {
+        // both columns' sums over the lane's rows for the rows of `rows` (with one decay per head: kept in `kept`)
+        auto contract = [&](const float (*rows)[CH], const Quad (&asked)[DR_GROUP][R4], Quad (*kept)[R4]) {
 #pragma unroll
             for (int i = 0; i < 2 * DR_GROUP; ++i) pairs[i] = 0;
+            if constexpr (CHANNEL) {
 #pragma unroll
-            for (int u = 0; u < R4; ++u) {
+                for (int u = 0; u < R4; ++u) {
 #pragma unroll
-                for (int i = 0; i < DR_GROUP; ++i) {
-                    pairs[2 * i] = fma2(S[0][u].a, m[i][u].a, pairs[2 * i]);
-                    pairs[2 * i + 1] = fma2(S[1][u].a, m[i][u].a, pairs[2 * i + 1]);
+                    for (int i = 0; i < DR_GROUP; ++i) {
+                        pairs[2 * i] = fma2(S[0][u].a, asked[i][u].a, pairs[2 * i]);
+                        pairs[2 * i + 1] = fma2(S[1][u].a, asked[i][u].a, pairs[2 * i + 1]);
+                    }
+#pragma unroll
+                    for (int i = 0; i < DR_GROUP; ++i) {
+                        pairs[2 * i] = fma2(S[0][u].b, asked[i][u].b, pairs[2 * i]);
+                        pairs[2 * i + 1] = fma2(S[1][u].b, asked[i][u].b, pairs[2 * i + 1]);
+                    }
                 }
+            } else {
 #pragma unroll
-                for (int i = 0; i < DR_GROUP; ++i) {
-                    pairs[2 * i] = fma2(S[0][u].b, m[i][u].b, pairs[2 * i]);
-                    pairs[2 * i + 1] = fma2(S[1][u].b, m[i][u].b, pairs[2 * i + 1]);
-                }
+                for (int i = 0; i < DR_GROUP; ++i)
+#pragma unroll
+                    for (int u = 0; u < R4; ++u) {
+                        const Quad m = load_quad(&rows[j0 + i][4 * (lane + DR_LANES * u)]);
+                        pairs[2 * i] = fma2(S[0][u].b, m.b, fma2(S[0][u].a, m.a, pairs[2 * i]));
+                        pairs[2 * i + 1] = fma2(S[1][u].b, m.b, fma2(S[1][u].a, m.a, pairs[2 * i + 1]));
+                        if (kept) kept[i][u] = m;
+                    }
             }
 #pragma unroll
             for (int i = 0; i < 2 * DR_GROUP; ++i) sums[i] = sum2(pairs[i]);
         };
-        ask(k, s.k);
+        Quad q[DR_GROUP][R4];
+        if constexpr (CHANNEL) ask(k, s.k);
         const float my_fade = CHANNEL ? 1.f : numbers[DR_FADE + own_i];
         const float my_v = s.v[j0 + own_i][c + own_x];
-        ask(q, s.q);
-        contract(k);
+        if constexpr (CHANNEL) ask(q, s.q);
+        contract(s.k, k, CHANNEL ? nullptr : k);
         // v - S^T k of the lane's own token and column, then its row of T times those of the group
         const float mine = fmaf(-my_fade, shared_sums<2 * DR_GROUP, DR_LANES>(sums), my_v);
-        contract(q);
+        contract(s.q, q, nullptr);
         if constexpr (CHANNEL) ask(k, s.k_end);
         float write[2] = {0.f, 0.f};
 #pragma unroll
