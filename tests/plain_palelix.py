@@ -223,6 +223,11 @@ def layer_runs(config):
     return runs + [(i, None) for i in range(stop, n)]
 
 
+def routed_runs(config):
+    """The numbers of the layer runs that route."""
+    return [run for run, (i, _) in enumerate(layer_runs(config)) if (config["layers"][i].get("mlp") or {}).get("kind") == "moe"]
+
+
 def forward(config, w, tokens, return_layers=False, forced=None, heard=None):
     """Logits [T, vocab] of one sequence. ``forced``: {number of the layer run: [T, top] expert choices}; ``heard``: a
     list that receives (own choice, margin) of every routed layer run."""
