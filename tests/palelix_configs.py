@@ -73,13 +73,14 @@ MODEL_B = model(128, 257, [
 ], loop=(1, 3, 2))
 
 # sizes that are multiples of nothing useful: width 100, an odd vocabulary, recurrent heads of 13 x 7 and 5 x 9, a convolution
-# of one tap and one of nine, no rotation, one expert, no repeated run
+# of one tap and one of nine, no rotation, one expert, no repeated run; an eps that keeps the norms of such small heads from
+# magnifying 16-bit rounding where a read-out is nearly zero
 MODEL_C = model(100, 131, [
     lightning(5, 13, 7, [0.8, 0.95, 0.0, 1.0, 0.6], mlp=moe(52, 10, 3)),
     parallel((5, 5, 12, 20, 0.4, None), (3, 1, 13, 7, 1), 1.3, 0.9, mlp=moe(36, 2, 2)),
     delta(5, 5, 5, 9, 9, mlp=moe(20, 1, 1)),
     parallel((3, 1, 17, 11, 0.5, (2, 50.0)), (2, 2, 6, 30, 2), 0.5, -1.1, mlp=dense(33)),
-])
+], eps=0.01)
 
 # recurrent layers only, so no paged cache at all, the whole model repeated
 MODEL_D = model(64, 97, [
