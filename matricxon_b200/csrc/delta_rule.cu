@@ -22,8 +22,8 @@
 //   decayed from the group's start, k'' to its end, G over the whole group, T and P 8 x 8. A first kernel forms them for
 //   all groups in parallel (decays enter as products of numbers up to one, nothing is divided); the second walks the
 //   groups: a block owns (sequence, head, 16 value columns), sixteen lanes share two columns with their rows in
-//   registers for the whole portion, so that a group costs one round of reductions (sixteen sums over sixteen lanes
-//   share their shuffles). Operands arrive in rounds by cp.async, two rounds ahead; products and sums are packed pairs of
+//   registers for the whole portion (8 columns and 32 lanes where blocks are few), so that a group costs one round of
+//   reductions (sixteen sums over sixteen lanes share their shuffles). Operands arrive in rounds by cp.async, two rounds ahead; products and sums are packed pairs of
 //   floats.
 // mx_delta_step: steps in which no sequence brings more than one token. A block owns (sequence, head): the state passes
 //   through registers once (a warp per group of value columns, a lane per four rows), reductions of sixteen columns
@@ -34,7 +34,7 @@
 
 namespace {
 
-constexpr int DR_COLS = 16, DR_LANES = 16, DR_THREADS = DR_COLS / 2 * DR_LANES;
+constexpr int DR_THREADS = 128;              // of a block of the scan
 constexpr int DR_GROUP = 8;                  // tokens of a group
 constexpr int DR_STAGES = 3;                 // rounds of the scan in shared memory: one computed, two on their way
 // a group's numbers: T and P (a row per token), the fades from its start to each token and from each token to its end
@@ -339,13 +339,13 @@ delta_groups_kernel(const DeltaParams p) {
     coef[DR_END + lane] = left;
 }
 
-// A round's operands. Sixteen lanes share two value columns, R4 groups of four rows a lane (dim <= 64 * R4): the rows
-// 4 (lane + 16 u), so that sixteen lanes' 16-byte loads are one contiguous row.
-template <int R4, int TOKENS, bool CHANNEL>
+// A round's operands. LANES lanes share two value columns, R4 groups of four rows a lane (dim <= 4 * LANES * R4): the rows
+// 4 (lane + LANES u), so that their 16-byte loads are one contiguous row.
+template <int LANES, int R4, int TOKENS, bool CHANNEL>
 struct ScanStage {
-    static constexpr int CH = 4 * DR_LANES * R4, GROUPS = TOKENS / DR_GROUP;
+    static constexpr int CH = 4 * LANES * R4, GROUPS = TOKENS / DR_GROUP, COLS = 2 * DR_THREADS / LANES;
     float k[TOKENS][CH], q[TOKENS][CH], k_end[CHANNEL ? TOKENS : 1][CHANNEL ? CH : 4], fade[CHANNEL ? GROUPS : 1][CHANNEL ? CH : 4];
-    float v[TOKENS][DR_COLS], coef[GROUPS][DR_COEF];
+    float v[TOKENS][COLS], coef[GROUPS][DR_COEF];
 };
 
 // Pairs of floats as the packed operations take them.
@@ -383,25 +383,26 @@ __device__ __forceinline__ Quad ask_quad(const float* p) {
     return v;
 }
 
-template <int R4, int TOKENS, bool CHANNEL>
+template <int LANES, int R4, int TOKENS, bool CHANNEL>
 __global__ void __launch_bounds__(DR_THREADS)
 delta_scan_kernel(const DeltaParams p) {
-    using Stage = ScanStage<R4, TOKENS, CHANNEL>;
+    using Stage = ScanStage<LANES, R4, TOKENS, CHANNEL>;
+    constexpr int COLS = Stage::COLS, PER = LANES / (2 * DR_GROUP);          // PER lanes hold the same sum of a group
     constexpr int CH = Stage::CH, ROW_THREADS = CH / 4, ROWS = DR_THREADS / ROW_THREADS;
     static_assert(DR_THREADS % ROW_THREADS == 0 && TOKENS % ROWS == 0, "a round's rows fill whole passes");
     extern __shared__ __align__(16) unsigned char scan_smem[];
     Stage* stages = reinterpret_cast<Stage*>(scan_smem);     // DR_STAGES rounds
     pdl_trigger();
-    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * DR_COLS, tid = threadIdx.x;
+    const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS, tid = threadIdx.x;
     const int t0 = p.cu_q[seq], t1 = p.cu_q[seq + 1];
     if (t1 <= t0) {
         // a padding sequence of a fixed-size batch, whose row bears its own number: defined output, no state
         pdl_wait();
-        if (seq >= t0 && tid < DR_COLS && col0 + tid < p.vdim)
+        if (seq >= t0 && tid < COLS && col0 + tid < p.vdim)
             p.out[((size_t)seq * p.heads + head) * p.vdim + col0 + tid] = 0.f;
         return;
     }
-    const int lane = tid & (DR_LANES - 1), c = 2 * (tid / DR_LANES), col = col0 + c;
+    const int lane = tid & (LANES - 1), c = 2 * (tid / LANES), col = col0 + c;
     const int group0 = group_of(t0, seq, 0);
     float* s_base = p.state + (size_t)p.state_slots[seq] * p.state_stride + p.state_offset + ((size_t)head * p.vdim + col) * p.dim;
     Quad S[2][R4];
@@ -409,7 +410,7 @@ delta_scan_kernel(const DeltaParams p) {
     for (int x = 0; x < 2; ++x)
 #pragma unroll
         for (int u = 0; u < R4; ++u) {
-            const int r = 4 * (lane + DR_LANES * u);
+            const int r = 4 * (lane + LANES * u);
             S[x][u] = col + x < p.vdim && r < p.dim ? load_quad(s_base + (size_t)x * p.dim + r) : Quad{0, 0};
         }
     if (p.dim < CH) {
@@ -447,8 +448,8 @@ delta_scan_kernel(const DeltaParams p) {
                     q_at += ROWS * row_stride;
                 }
             }
-            if (tid < TOKENS * (DR_COLS / 4)) {
-                const int j = tid / (DR_COLS / 4), e = (tid % (DR_COLS / 4)) * 4;
+            if (tid < TOKENS * (COLS / 4)) {
+                const int j = tid / (COLS / 4), e = (tid % (COLS / 4)) * 4;
                 const bool live = base + j < n && col0 + e < p.vdim;
                 copy16(&s.v[j][e], live ? v_from + (size_t)(base + j) * p.channels + e : v_from, live);
             }
@@ -465,8 +466,8 @@ delta_scan_kernel(const DeltaParams p) {
         copies_commit();
     };
     // the one of the group's sums that a lane ends up with: token own_i, column own_x
-    const int own_i = lane >> 1, own_x = lane & 1;
-    const bool writes = col + own_x < p.vdim;
+    const int own_i = lane / (2 * PER), own_x = lane / PER & 1;
+    const bool writes = lane % PER == 0 && col + own_x < p.vdim;
     const size_t out_stride = (size_t)p.heads * p.vdim;
     float* out = p.out + ((size_t)(t0 + own_i) * p.heads + head) * p.vdim + col + own_x;
     auto advance = [&](const Stage& s, int g, int t) {
@@ -479,7 +480,7 @@ delta_scan_kernel(const DeltaParams p) {
 #pragma unroll
             for (int i = 0; i < DR_GROUP; ++i)
 #pragma unroll
-                for (int u = 0; u < R4; ++u) into[i][u] = ask_quad(&rows[j0 + i][4 * (lane + DR_LANES * u)]);
+                for (int u = 0; u < R4; ++u) into[i][u] = ask_quad(&rows[j0 + i][4 * (lane + LANES * u)]);
         };
         // both columns' sums over the lane's rows for the rows of `rows` (with one decay per head: kept in `kept`)
         auto contract = [&](const float (*rows)[CH], const Quad (&asked)[DR_GROUP][R4], Quad (*kept)[R4]) {
@@ -504,7 +505,7 @@ delta_scan_kernel(const DeltaParams p) {
                 for (int i = 0; i < DR_GROUP; ++i)
 #pragma unroll
                     for (int u = 0; u < R4; ++u) {
-                        const Quad m = load_quad(&rows[j0 + i][4 * (lane + DR_LANES * u)]);
+                        const Quad m = load_quad(&rows[j0 + i][4 * (lane + LANES * u)]);
                         pairs[2 * i] = fma2(S[0][u].b, m.b, fma2(S[0][u].a, m.a, pairs[2 * i]));
                         pairs[2 * i + 1] = fma2(S[1][u].b, m.b, fma2(S[1][u].a, m.a, pairs[2 * i + 1]));
                         if (kept) kept[i][u] = m;
@@ -520,26 +521,26 @@ delta_scan_kernel(const DeltaParams p) {
         if constexpr (CHANNEL) ask(q, s.q);
         contract(s.k, k, CHANNEL ? nullptr : k);
         // v - S^T k of the lane's own token and column, then its row of T times those of the group
-        const float mine = fmaf(-my_fade, shared_sums<2 * DR_GROUP, DR_LANES>(sums), my_v);
+        const float mine = fmaf(-my_fade, shared_sums<2 * DR_GROUP, LANES>(sums), my_v);
         contract(s.q, q, nullptr);
         if constexpr (CHANNEL) ask(k, s.k_end);
         float write[2] = {0.f, 0.f};
 #pragma unroll
         for (int j = 0; j < DR_GROUP; j += 4) {
             const float4 row = *reinterpret_cast<const float4*>(&numbers[own_i * DR_GROUP + j]);
-            write[0] = fmaf(row.x, __shfl_sync(0xffffffffu, mine, 2 * j + own_x, DR_LANES), write[0]);
-            write[1] = fmaf(row.y, __shfl_sync(0xffffffffu, mine, 2 * j + 2 + own_x, DR_LANES), write[1]);
-            write[0] = fmaf(row.z, __shfl_sync(0xffffffffu, mine, 2 * j + 4 + own_x, DR_LANES), write[0]);
-            write[1] = fmaf(row.w, __shfl_sync(0xffffffffu, mine, 2 * j + 6 + own_x, DR_LANES), write[1]);
+            write[0] = fmaf(row.x, __shfl_sync(0xffffffffu, mine, PER * (2 * j + own_x), LANES), write[0]);
+            write[1] = fmaf(row.y, __shfl_sync(0xffffffffu, mine, PER * (2 * j + 2 + own_x), LANES), write[1]);
+            write[0] = fmaf(row.z, __shfl_sync(0xffffffffu, mine, PER * (2 * j + 4 + own_x), LANES), write[0]);
+            write[1] = fmaf(row.w, __shfl_sync(0xffffffffu, mine, PER * (2 * j + 6 + own_x), LANES), write[1]);
         }
         const float my_write = write[0] + write[1];
         float w[DR_GROUP][2];
 #pragma unroll
         for (int i = 0; i < DR_GROUP; ++i) {
-            w[i][0] = __shfl_sync(0xffffffffu, my_write, 2 * i, DR_LANES);
-            w[i][1] = __shfl_sync(0xffffffffu, my_write, 2 * i + 1, DR_LANES);
+            w[i][0] = __shfl_sync(0xffffffffu, my_write, PER * 2 * i, LANES);
+            w[i][1] = __shfl_sync(0xffffffffu, my_write, PER * (2 * i + 1), LANES);
         }
-        const float my_seen = shared_sums<2 * DR_GROUP, DR_LANES>(sums);
+        const float my_seen = shared_sums<2 * DR_GROUP, LANES>(sums);
         // o = S^T q + P u
         float o[2] = {my_fade * my_seen, 0.f};
 #pragma unroll
@@ -567,7 +568,7 @@ delta_scan_kernel(const DeltaParams p) {
         } else {
 #pragma unroll
             for (int u = 0; u < R4; ++u) {
-                const Quad f = load_quad(&s.fade[CHANNEL ? g : 0][CHANNEL ? 4 * (lane + DR_LANES * u) : 0]);
+                const Quad f = load_quad(&s.fade[CHANNEL ? g : 0][CHANNEL ? 4 * (lane + LANES * u) : 0]);
 #pragma unroll
                 for (int x = 0; x < 2; ++x) S[x][u] = {mul2(S[x][u].a, f.a), mul2(S[x][u].b, f.b)};
             }
@@ -598,7 +599,7 @@ delta_scan_kernel(const DeltaParams p) {
     for (int x = 0; x < 2; ++x)
 #pragma unroll
         for (int u = 0; u < R4; ++u) {
-            const int r = 4 * (lane + DR_LANES * u);
+            const int r = 4 * (lane + LANES * u);
             if (col + x < p.vdim && r < p.dim)
                 *reinterpret_cast<ulonglong2*>(s_base + (size_t)x * p.dim + r) = make_ulonglong2(S[x][u].a, S[x][u].b);
         }
@@ -718,29 +719,35 @@ void launch_prepare(const PrepareParams& p, cudaStream_t stream) {
         mx_launch_chained(delta_prepare_kernel<TAPS, 8, NV>, dim3((p.n_tokens + 7) / 8, (items + 3) / 4), dim3(128), 0, stream, p);
 }
 
-template <int R4, int TOKENS, bool CHANNEL>
-int launch_scan(const DeltaParams& p, int n_seqs, cudaStream_t stream) {
-    constexpr size_t smem = DR_STAGES * sizeof(ScanStage<R4, TOKENS, CHANNEL>);
+template <int LANES, int R4, int TOKENS, bool CHANNEL>
+int launch_walk(const DeltaParams& p, int n_seqs, cudaStream_t stream) {
+    constexpr size_t smem = DR_STAGES * sizeof(ScanStage<LANES, R4, TOKENS, CHANNEL>);
+    constexpr int COLS = ScanStage<LANES, R4, TOKENS, CHANNEL>::COLS;
     static bool ready = false;
     if (!ready) {
-        if (cudaFuncSetAttribute(delta_scan_kernel<R4, TOKENS, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        if (cudaFuncSetAttribute(delta_scan_kernel<LANES, R4, TOKENS, CHANNEL>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)smem) != cudaSuccess)
             MX_REFUSE("delta rule: cannot reserve %zu bytes of shared memory", smem);
         ready = true;
     }
-    const dim3 grid(p.n_tokens, (p.heads + 3) / 4);
-    if (p.dim <= 128) mx_launch_chained(delta_groups_kernel<1, CHANNEL>, grid, dim3(128), 0, stream, p);
-    else mx_launch_chained(delta_groups_kernel<2, CHANNEL>, grid, dim3(128), 0, stream, p);
-    mx_launch_chained(delta_scan_kernel<R4, TOKENS, CHANNEL>, dim3(n_seqs, p.heads, (p.vdim + DR_COLS - 1) / DR_COLS),
+    mx_launch_chained(delta_scan_kernel<LANES, R4, TOKENS, CHANNEL>, dim3(n_seqs, p.heads, (p.vdim + COLS - 1) / COLS),
                       dim3(DR_THREADS), smem, stream, p);
     return mx_launch_status();
 }
 
 template <bool CHANNEL>
-int pick_scan(const DeltaParams& p, int n_seqs, cudaStream_t stream) {
-    if (p.dim <= 64) return launch_scan<1, 16, CHANNEL>(p, n_seqs, stream);
-    if (p.dim <= 128) return launch_scan<2, 16, CHANNEL>(p, n_seqs, stream);
-    return launch_scan<4, 8, CHANNEL>(p, n_seqs, stream);
+int launch_scan(const DeltaParams& p, int n_seqs, int sms, cudaStream_t stream) {
+    const dim3 grid(p.n_tokens, (p.heads + 3) / 4);
+    if (p.dim <= 128) mx_launch_chained(delta_groups_kernel<1, CHANNEL>, grid, dim3(128), 0, stream, p);
+    else mx_launch_chained(delta_groups_kernel<2, CHANNEL>, grid, dim3(128), 0, stream, p);
+    // few columns: twice as many lanes to a column shorten each walk, as long as no SM gets two of the then twice as many
+    // blocks (2,048 tokens x 8 heads of 128 x 128: 218 -> 196 us; at 16 heads 224 -> 251)
+    const long long blocks = (long long)n_seqs * p.heads * ((p.vdim + 15) / 16);
+    const bool wide = p.dim > 64 && 2 * blocks <= sms;
+    if (p.dim <= 64) return launch_walk<16, 1, 16, CHANNEL>(p, n_seqs, stream);
+    if (p.dim <= 128)
+        return wide ? launch_walk<32, 1, 16, CHANNEL>(p, n_seqs, stream) : launch_walk<16, 2, 16, CHANNEL>(p, n_seqs, stream);
+    return wide ? launch_walk<32, 2, 8, CHANNEL>(p, n_seqs, stream) : launch_walk<16, 4, 8, CHANNEL>(p, n_seqs, stream);
 }
 
 const char* delta_sizes(int qk_heads, int heads, int dim, int vdim) {
@@ -824,7 +831,13 @@ extern "C" int mx_delta_scan(const float* qkv, const float* beta, const float* d
     p.tok_seq = tok_seq; p.out = out; p.n_tokens = n_tokens; p.coef = scratch;
     p.group_decay = scratch + groups * heads * DR_COEF;
     p.decayed = p.group_decay + groups * heads * dim;
-    return per_channel ? pick_scan<true>(p, n_seqs, stream) : pick_scan<false>(p, n_seqs, stream);
+    static int sms = 0;
+    if (sms == 0) {
+        int device = 0;
+        cudaGetDevice(&device);
+        cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
+    }
+    return per_channel ? launch_scan<true>(p, n_seqs, sms, stream) : launch_scan<false>(p, n_seqs, sms, stream);
 }
 
 // The scan of steps without a sequence of more than one token, with what follows it:

@@ -204,7 +204,7 @@ def plain_delta(qkv, beta, g, heads, kv, dim, vdim):
 
 @pytest.mark.parametrize("channel", [False, True])
 @pytest.mark.parametrize("heads, kv, dim, vdim", [(3, 3, 20, 28), (4, 2, 64, 128), (2, 1, 128, 64), (6, 2, 12, 20), (1, 1, 96, 24),
-                                                  (2, 2, 160, 40), (4, 1, 256, 16), (5, 5, 8, 8)])
+                                                  (2, 2, 160, 40), (4, 1, 256, 16), (5, 5, 8, 8), (16, 4, 128, 128), (8, 8, 256, 64)])
 def test_delta_rule_kernels(heads, kv, dim, vdim, channel):
     """Portions through the groups of eight (whole groups, one token more and less, single tokens among them), from and to
     slots, then single tokens through the step kernel, which ends in norm, weight and gate."""
